@@ -1257,6 +1257,272 @@ class PetanexConfig(ModelConfig):
         return out
 
 
+@dataclass(frozen=True)
+class SelectiveScanConfig:
+    """A selective scan: ``inner`` channels with ``state`` states each, step sizes through ``dt_rank`` values, a
+    convolution of ``conv`` taps."""
+
+    inner: int
+    state: int
+    dt_rank: int
+    conv: int
+
+    @staticmethod
+    def parse(m: Mapping[str, Any], where: str) -> "SelectiveScanConfig":
+        return SelectiveScanConfig(**{key: _count(m, key, where) for key in ("inner", "state", "dt_rank", "conv")})
+
+    def to_json_dict(self) -> Dict[str, Any]:
+        return {"inner": self.inner, "state": self.state, "dt_rank": self.dt_rank, "conv": self.conv}
+
+
+@dataclass(frozen=True)
+class GatedLinearConfig:
+    """Gated linear attention: ``heads`` heads of ``dim`` key and ``vdim`` value channels, decays to the power of
+    ``1 / tau``."""
+
+    heads: int
+    dim: int
+    vdim: int
+    tau: float
+
+    @staticmethod
+    def parse(m: Mapping[str, Any], where: str) -> "GatedLinearConfig":
+        tau = _number(m, "tau", where)
+        if not tau > 0:
+            raise ConfigError(f"{where}: tau={tau} must be positive")
+        return GatedLinearConfig(heads=_count(m, "heads", where), dim=_count(m, "dim", where),
+                                 vdim=_count(m, "vdim", where), tau=tau)
+
+    def to_json_dict(self) -> Dict[str, Any]:
+        return {"heads": self.heads, "dim": self.dim, "vdim": self.vdim, "tau": self.tau}
+
+
+@dataclass(frozen=True)
+class LongWaveRotation:
+    """Rotation of the first ``dims`` dims of a head; ``scaling`` (None: none) stretches pairs of long wavelengths:
+    (factor, low, high, original)."""
+
+    base: float
+    dims: int
+    scaling: Optional[Tuple[float, float, float, float]] = None
+
+    @staticmethod
+    def parse(m: Mapping[str, Any], where: str) -> "LongWaveRotation":
+        dims = _count(m, "dims", where)
+        if dims % 2:
+            raise ConfigError(f"{where}: dims={dims} must be even")
+        scaling = None
+        if m.get("scaling") is not None:
+            raw = _mapping(m, "scaling", where)
+            scaling = tuple(_number(raw, key, where + ".scaling") for key in ("factor", "low", "high", "original"))
+            factor, low, high, original = scaling
+            if factor <= 0 or low <= 0 or original <= 0 or high < low:
+                raise ConfigError(f"{where}.scaling: factor, low and original must be positive and high at least low")
+        return LongWaveRotation(base=_number(m, "base", where), dims=dims, scaling=scaling)
+
+    def to_json_dict(self) -> Dict[str, Any]:
+        out: Dict[str, Any] = {"base": self.base, "dims": self.dims}
+        if self.scaling is not None:
+            out["scaling"] = dict(zip(("factor", "low", "high", "original"), self.scaling))
+        return out
+
+
+@dataclass(frozen=True)
+class NormedAttentionConfig:
+    """Causal attention with queries and keys normed over the whole projection; ``kv_from``: the layer whose cached keys
+    and values it reads (None: its own)."""
+
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    rot: Optional[LongWaveRotation] = None
+    kv_from: Optional[int] = None
+
+    @staticmethod
+    def parse(m: Mapping[str, Any], where: str) -> "NormedAttentionConfig":
+        heads, kv_heads = _count(m, "heads", where), _count(m, "kv_heads", where)
+        if heads % kv_heads:
+            raise ConfigError(f"{where}: heads={heads} must be a multiple of kv_heads={kv_heads}")
+        for key in ("mask", "sink", "window"):
+            if m.get(key):
+                raise ConfigError(f"{where}: {key!r} is not a key of this mixer")
+        dim = _count(m, "dim", where)
+        rot = None
+        if m.get("rot") is not None:
+            rot = LongWaveRotation.parse(_mapping(m, "rot", where), where + ".rot")
+            if rot.dims > dim:
+                raise ConfigError(f"{where}.rot: dims={rot.dims} is more than dim={dim}")
+        kv_from = m.get("kv_from")
+        if kv_from is not None and (isinstance(kv_from, bool) or not isinstance(kv_from, int) or kv_from < 0):
+            raise ConfigError(f"{where}: kv_from must name an earlier layer, got {kv_from!r}")
+        return NormedAttentionConfig(heads=heads, kv_heads=kv_heads, dim=dim, vdim=_count(m, "vdim", where),
+                                     scale=_number(m, "scale", where), rot=rot, kv_from=kv_from)
+
+    def to_json_dict(self) -> Dict[str, Any]:
+        out: Dict[str, Any] = {"heads": self.heads, "kv_heads": self.kv_heads, "dim": self.dim, "vdim": self.vdim,
+                               "scale": self.scale}
+        if self.rot is not None:
+            out["rot"] = self.rot.to_json_dict()
+        if self.kv_from is not None:
+            out["kv_from"] = self.kv_from
+        return out
+
+
+@dataclass(frozen=True)
+class SoftmaxExpertsConfig:
+    """``experts`` gated feed-forwards of inner width ``ff``, ``top`` of them per token, weighted by the softmax over the
+    chosen router logits."""
+
+    experts: int
+    top: int
+    ff: int
+
+    @staticmethod
+    def parse(m: Mapping[str, Any], where: str) -> "SoftmaxExpertsConfig":
+        if m.get("kind") != "moe":
+            raise ConfigError(f"{where}: mlp kind {m.get('kind')!r} is not supported ('moe' is)")
+        if m.get("shared"):
+            raise ConfigError(f"{where}: 'shared' is not a key of this feed-forward")
+        router = _mapping(m, "router", where)
+        experts, top = _count(router, "experts", where + ".router"), _count(router, "top", where + ".router")
+        if top > experts:
+            raise ConfigError(f"{where}.router: top={top} is more than experts={experts}")
+        return SoftmaxExpertsConfig(experts=experts, top=top,
+                                    ff=_count(_mapping(m, "expert", where), "ff", where + ".expert"))
+
+    def to_json_dict(self) -> Dict[str, Any]:
+        return {"kind": "moe", "expert": {"ff": self.ff}, "router": {"experts": self.experts, "top": self.top}}
+
+
+@dataclass(frozen=True)
+class BigramConfig:
+    """A second embedding by (previous token, token): row (previous * mul_prev + token * mul_cur) mod buckets."""
+
+    buckets: int
+    mul_prev: int
+    mul_cur: int
+
+    @staticmethod
+    def parse(m: Mapping[str, Any], where: str) -> "BigramConfig":
+        values = {}
+        for key in ("mul_prev", "mul_cur"):
+            value = _require(m, key)
+            if isinstance(value, bool) or not isinstance(value, int):
+                raise ConfigError(f"{where}: {key} must be an integer, got {value!r}")
+            values[key] = value
+        return BigramConfig(buckets=_count(m, "buckets", where), **values)
+
+    def to_json_dict(self) -> Dict[str, Any]:
+        return {"buckets": self.buckets, "mul_prev": self.mul_prev, "mul_cur": self.mul_cur}
+
+
+@dataclass(frozen=True)
+class DemavikLayerConfig:
+    """``type`` mamba1: ``scan``; gla: ``linear``; attention: ``attention``."""
+
+    type: str
+    scan: Optional[SelectiveScanConfig] = None
+    linear: Optional[GatedLinearConfig] = None
+    attention: Optional[NormedAttentionConfig] = None
+    mlp: Optional[SoftmaxExpertsConfig] = None
+
+    def mixer_json_dict(self) -> Dict[str, Any]:
+        return (self.scan or self.linear or self.attention).to_json_dict()
+
+
+@dataclass(frozen=True)
+class DemavikConfig(ModelConfig):
+    """``Demavik``: norms on the sublayers' results, times a constant, before they join the stream; the mixer is a selective
+    scan (``mamba1``), gated linear attention (``gla``) or causal attention (``attention``), which may read another
+    layer's cached keys and values; the feed-forward is routed experts or nothing; the embedding adds a row by
+    the pair of tokens.  config.json keys: ``vocab``, ``width``, ``norm.eps``, ``residual_mult``, ``embedding`` ({scale,
+    bigram}) and ``layers`` (a list of ``{type, mixer, mlp}``)."""
+
+    layers: Tuple[DemavikLayerConfig, ...] = ()
+    norm_eps: float = 1e-5
+    residual_mult: float = 1.0
+    embedding_scale: float = 1.0
+    bigram: Optional[BigramConfig] = None
+    torch_dtype: str = "bfloat16"
+
+    @staticmethod
+    def from_dict(cfg: Mapping[str, Any]) -> "DemavikConfig":
+        name = cfg.get("architecture") or (cfg.get("architectures") or ["Demavik"])[0]
+        raw_layers = cfg.get("layers")
+        if not isinstance(raw_layers, (list, tuple)) or not raw_layers:
+            raise ConfigError("config.json key 'layers' must be a non-empty list")
+        layers = []
+        for index, raw in enumerate(raw_layers):
+            where = f"config.json layers[{index}]"
+            if not isinstance(raw, Mapping):
+                raise ConfigError(f"{where} must be an object")
+            kind = raw.get("type")
+            m, at = _mapping(raw, "mixer", where), where + ".mixer"
+            mlp = None
+            if raw.get("mlp") is not None:
+                mlp = SoftmaxExpertsConfig.parse(_mapping(raw, "mlp", where), where + ".mlp")
+            if kind == "mamba1":
+                layer = DemavikLayerConfig(type=kind, scan=SelectiveScanConfig.parse(m, at), mlp=mlp)
+            elif kind == "gla":
+                layer = DemavikLayerConfig(type=kind, linear=GatedLinearConfig.parse(m, at), mlp=mlp)
+            elif kind == "attention":
+                layer = DemavikLayerConfig(type=kind, attention=NormedAttentionConfig.parse(m, at), mlp=mlp)
+            else:
+                raise ConfigError(f"{where}: layer type {kind!r} is not supported ('mamba1', 'gla' and 'attention' are)")
+            source = None if layer.attention is None else layer.attention.kv_from
+            if source is not None:
+                other = layers[source].attention if source < index else None
+                if other is None or other.kv_from is not None:
+                    raise ConfigError(f"{at}: kv_from={source} must name an earlier attention layer with keys of its own")
+                mine = layer.attention
+                if (mine.kv_heads, mine.dim, mine.vdim) != (other.kv_heads, other.dim, other.vdim):
+                    raise ConfigError(f"{at}: kv_heads, dim and vdim must be those of layer {source}, whose keys it reads")
+            layers.append(layer)
+        scale, bigram = 1.0, None
+        if cfg.get("embedding") is not None:
+            embedding = _mapping(cfg, "embedding", "config.json")
+            scale = _number(embedding, "scale", "config.json embedding") if embedding.get("scale") is not None else 1.0
+            if embedding.get("bigram") is not None:
+                bigram = BigramConfig.parse(_mapping(embedding, "bigram", "config.json embedding"),
+                                            "config.json embedding.bigram")
+        eos = cfg.get("eos_token_id")
+        eos_ids: Tuple[int, ...] = () if eos is None else ((eos,) if isinstance(eos, int) else tuple(int(t) for t in eos))
+        return DemavikConfig(
+            architecture=str(name),
+            vocab_size=_count(cfg, "vocab", "config.json"),
+            hidden_size=_count(cfg, "width", "config.json"),
+            num_hidden_layers=len(layers),
+            max_position_embeddings=int(cfg.get("max_position_embeddings", 1 << 20)),
+            tie_word_embeddings=False,
+            eos_token_ids=eos_ids,
+            layers=tuple(layers),
+            norm_eps=_number(_mapping(cfg, "norm", "config.json"), "eps", "config.json norm"),
+            residual_mult=_number(cfg, "residual_mult", "config.json") if cfg.get("residual_mult") is not None else 1.0,
+            embedding_scale=scale,
+            bigram=bigram,
+            torch_dtype=str(cfg.get("torch_dtype", "bfloat16")),
+        )
+
+    def to_json_dict(self) -> Dict[str, Any]:
+        embedding: Dict[str, Any] = {"scale": self.embedding_scale}
+        if self.bigram is not None:
+            embedding["bigram"] = self.bigram.to_json_dict()
+        out: Dict[str, Any] = {
+            "architecture": self.architecture, "vocab": self.vocab_size, "width": self.hidden_size,
+            "norm": {"eps": self.norm_eps}, "residual_mult": self.residual_mult, "embedding": embedding,
+            "layers": [{"type": layer.type, "mixer": layer.mixer_json_dict(),
+                        "mlp": None if layer.mlp is None else layer.mlp.to_json_dict()} for layer in self.layers],
+            "torch_dtype": self.torch_dtype,
+        }
+        if self.max_position_embeddings != 1 << 20:
+            out["max_position_embeddings"] = self.max_position_embeddings
+        if self.eos_token_ids:
+            out["eos_token_id"] = list(self.eos_token_ids)
+        return out
+
+
 def read_config_json(model_dir: str) -> Dict[str, Any]:
     path = os.path.join(model_dir, "config.json")
     if not os.path.isfile(path):

@@ -4,7 +4,7 @@ There are four libraries: ``core`` (row-wise kernels, sampling, GEMMs; one build
 ``attention`` (one build per head size, ``-DVX_HEAD_DIM=<D>``), ``mixers`` (recurrent mixers,
 the delta rule among them, and expert feed-forwards; one build) and ``heads`` (token shift, the
 input convolution, differential attention's two ends, the gated activations; one build), so a process compiles what its model needs and
-nothing else.  A build is keyed by a hash of its sources, flags and compiler
+nothing else.  A build is keyed by a hash of its sources, the headers they include, flags and compiler
 version; it is made once and reused.  Builds go to ``velox_b200/_build`` inside the package when
 that is writable, else to ``$VELOX_B200_BUILD_DIR``, else to a per-user folder under the
 system's temporary directory.  nvcc cross-compiles without a GPU, so the build also runs on a
@@ -39,11 +39,10 @@ if os.environ.get("VELOX_B200_TRACE") == "1":
 CORE_SOURCES = ("core.cu", "sampling.cu", "gemm_bf16.cu", "residual.cu", "latent.cu")
 # Mixers with a state of fixed size per request and feed-forwards with experts: built only for
 # models that have such parts.
-MIXER_SOURCES = ("sequence.cu", "delta_rule.cu", "gated_delta.cu", "routed.cu")
+MIXER_SOURCES = ("sequence.cu", "delta_rule.cu", "gated_delta.cu", "gated_linear.cu", "selective.cu", "routed.cu")
 # Row kernels around attention heads and gated feed-forwards: built for models with such parts.
 HEADS_SOURCES = ("heads.cu",)
 ATTENTION_SOURCES = ("attention.cu",)
-HEADERS = ("common.cuh", "recurrent.cuh", "delta_rule.cuh", "attention_static.h")
 
 _loaded: Dict[str, ctypes.CDLL] = {}
 _lock = threading.Lock()
@@ -98,9 +97,22 @@ def _nvcc_version(nvcc: str) -> str:
     return out.strip().splitlines()[-1]
 
 
+def _included(sources: Sequence[str]) -> List[str]:
+    """The headers of this directory that the sources include, directly or through one another."""
+    found: List[str] = []
+    waiting = list(sources)
+    while waiting:
+        with open(os.path.join(_SRC_DIR, waiting.pop()), "r", encoding="utf-8") as handle:
+            for name in re.findall(r'^\s*#include\s+"([^"]+)"', handle.read(), re.MULTILINE):
+                if name not in found:
+                    found.append(name)
+                    waiting.append(name)
+    return sorted(found)
+
+
 def _build_key(sources: Sequence[str], defines: Sequence[str], nvcc_version: str) -> str:
     digest = hashlib.sha256()
-    for name in list(sources) + list(HEADERS):
+    for name in list(sources) + _included(sources):
         with open(os.path.join(_SRC_DIR, name), "rb") as handle:
             digest.update(name.encode())
             digest.update(handle.read())

@@ -140,6 +140,24 @@ __device__ __forceinline__ void bulk_copy_g2s(uint32_t dst, const void* src, uin
 }
 
 // ---------------------------------------------------------------------------------------------
+// Distributed shared memory: the address of `local` in the CTA of another rank of the cluster, a store there, and
+// the cluster's barrier.
+// ---------------------------------------------------------------------------------------------
+__device__ __forceinline__ uint32_t peer_address(const void* local, uint32_t rank) {
+  const uint32_t addr = smem_u32(local);
+  uint32_t remote;
+  asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(remote) : "r"(addr), "r"(rank));
+  return remote;
+}
+__device__ __forceinline__ void store_peer(uint32_t remote, float v) {
+  asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(remote), "f"(v) : "memory");
+}
+__device__ __forceinline__ void cluster_meet() {
+  asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
+  asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
+}
+
+// ---------------------------------------------------------------------------------------------
 // Programmatic dependent launch.  Every kernel of a step is launched with the attribute that
 // lets it start while its predecessor in the stream is still running; it may then do work that
 // does not depend on the predecessor (set up barriers, prefetch weights) and must call
@@ -173,6 +191,31 @@ inline cudaError_t launch_pdl(void (*kernel)(KArgs...), dim3 grid, dim3 block, s
   attribute[0].val.programmaticStreamSerializationAllowed = 1;
   config.attrs = attribute;
   config.numAttrs = serialised ? 0 : 1;
+  return cudaLaunchKernelEx(&config, kernel, static_cast<KArgs>(args)...);
+}
+
+// The same with the grid's x cut into clusters of `cluster` CTAs.
+template <typename... KArgs, typename... Args>
+inline cudaError_t launch_pdl_cluster(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem, int cluster,
+                                      cudaStream_t stream, Args&&... args) {
+  cudaLaunchConfig_t config = {};
+  config.gridDim = grid;
+  config.blockDim = block;
+  config.dynamicSmemBytes = smem;
+  config.stream = stream;
+  static const bool serialised = [] {
+    const char* value = getenv("VELOX_B200_NO_PDL");
+    return value != nullptr && value[0] == '1';
+  }();
+  cudaLaunchAttribute attributes[2];
+  attributes[0].id = cudaLaunchAttributeClusterDimension;
+  attributes[0].val.clusterDim.x = (unsigned)cluster;
+  attributes[0].val.clusterDim.y = 1;
+  attributes[0].val.clusterDim.z = 1;
+  attributes[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+  attributes[1].val.programmaticStreamSerializationAllowed = 1;
+  config.attrs = attributes;
+  config.numAttrs = serialised ? 1 : 2;
   return cudaLaunchKernelEx(&config, kernel, static_cast<KArgs>(args)...);
 }
 

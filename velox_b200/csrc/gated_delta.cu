@@ -50,58 +50,6 @@ __device__ __forceinline__ void block_sum3(float& a, float& b, float& c, float* 
   for (int w = 0; w < GD_THREADS / 32; ++w) a += scratch[3 * w], b += scratch[3 * w + 1], c += scratch[3 * w + 2];
 }
 
-// out[n] = sum over r of w[n][r] * v[r] for n < count, v in shared memory: groups of lanes share a row
-// (16-byte packs where `packs` says that every row starts on one and holds whole ones), the loads of
-// four rows of a group under way together.
-template <typename T>
-__device__ __forceinline__ void rank_product(const T* __restrict__ w, const float* __restrict__ v, int rank, int count,
-                                             bool packs, float* __restrict__ out) {
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  constexpr int WARPS = GD_THREADS / 32, PK = 16 / (int)sizeof(T);
-  int lanes = 32;
-  if (packs)
-    while (lanes > 1 && (lanes / 2) * PK >= rank) lanes /= 2;
-  const int groups = 32 / lanes, sub = lane & (lanes - 1), mine = warp * groups + lane / lanes;
-  const int stride = WARPS * groups;
-  for (int n0 = mine; n0 - mine < count; n0 += 4 * stride) {
-    float acc[4] = {0.f, 0.f, 0.f, 0.f};
-    if (packs) {
-      for (int r = sub * PK; r < rank; r += lanes * PK) {
-        uint4 raw[4];
-#pragma unroll
-        for (int u = 0; u < 4; ++u) {
-          const int n = n0 + u * stride;
-          raw[u] = n < count ? *reinterpret_cast<const uint4*>(w + (size_t)n * rank + r) : make_uint4(0u, 0u, 0u, 0u);
-        }
-#pragma unroll
-        for (int u = 0; u < 4; ++u) {
-          const T* e = reinterpret_cast<const T*>(&raw[u]);
-#pragma unroll
-          for (int q = 0; q < PK; ++q) acc[u] = fmaf(to_float(e[q]), v[r + q], acc[u]);
-        }
-      }
-    } else {
-      for (int r = sub; r < rank; r += lanes) {
-        const float vr = v[r];
-#pragma unroll
-        for (int u = 0; u < 4; ++u) {
-          const int n = n0 + u * stride;
-          if (n < count) acc[u] = fmaf(to_float(w[(size_t)n * rank + r]), vr, acc[u]);
-        }
-      }
-    }
-    for (int off = lanes / 2; off > 0; off >>= 1) {
-#pragma unroll
-      for (int u = 0; u < 4; ++u) acc[u] += __shfl_xor_sync(0xffffffffu, acc[u], off);
-    }
-    if (sub == 0) {
-#pragma unroll
-      for (int u = 0; u < 4; ++u)
-        if (n0 + u * stride < count) out[n0 + u * stride] = acc[u];
-    }
-  }
-}
-
 template <typename T, int FORM, int RL, int NCH, bool VEC>
 __global__ void __launch_bounds__(GD_THREADS)
 gated_delta_step_kernel(GatedDelta p, GatedDeltaOut o, float* __restrict__ state, long long state_stride,
@@ -181,12 +129,12 @@ gated_delta_step_kernel(GatedDelta p, GatedDeltaOut o, float* __restrict__ state
   if (FORM == DR_CHANNEL) {
     if (o.rank_a > 0) {
       const bool packs = o.rank_a % (16 / (int)sizeof(T)) == 0;
-      rank_product<T>((const T*)o.a_up + (size_t)h * Dk * o.rank_a, low_a, o.rank_a, Dk, packs, w_s);
+      rank_product<T, GD_THREADS / 32>((const T*)o.a_up + (size_t)h * Dk * o.rank_a, low_a, o.rank_a, Dk, packs, w_s);
     }
   }
   if (o.rank_g > 0) {
     const bool packs = o.rank_g % (16 / (int)sizeof(T)) == 0;
-    rank_product<T>((const T*)o.g_up + (size_t)h * Dv * o.rank_g, low_g, o.rank_g, Dv, packs, gate_s);
+    rank_product<T, GD_THREADS / 32>((const T*)o.g_up + (size_t)h * Dv * o.rank_g, low_g, o.rank_g, Dv, packs, gate_s);
   } else {
     for (int c = tid; c < Dv; c += GD_THREADS) gate_s[c] = to_float(gate_row[(size_t)h * Dv + c]);
   }

@@ -19,6 +19,8 @@
 //   token_gate_kernel        gelu(s[t, :]) * a column range of row `token id` of a table
 //   token_input_kernel       the whole of a layer's token input for a few tokens, a cluster of CTAs
 //                            per token: g = gelu(W_gate x) * table row, y = W_proj g, x += rms(y) * w
+//   embed_pairs_kernel       embedding plus a second table's row for (previous token, token)
+//   norm_rope_store_kernel   q and k normed over the whole projection, rotated, k and v to the cache
 //
 // Everything between the loads and the stores is float32.  Every sum has an order that depends
 // on the sizes only.
@@ -901,20 +903,6 @@ __global__ void token_gate_kernel(const T* __restrict__ s, long long s_stride, c
 // columns beyond dim are zero), width a multiple of 8.
 constexpr int TI_CLUSTER = 8, TI_THREADS = 256;
 
-__device__ __forceinline__ uint32_t peer_address(const void* local, uint32_t rank) {
-  const uint32_t addr = smem_u32(local);
-  uint32_t remote;
-  asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(remote) : "r"(addr), "r"(rank));
-  return remote;
-}
-__device__ __forceinline__ void store_peer(uint32_t remote, float v) {
-  asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(remote), "f"(v) : "memory");
-}
-__device__ __forceinline__ void cluster_meet() {
-  asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
-  asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
-}
-
 __device__ __forceinline__ void ti_copy_16(__nv_bfloat16* dst, const __nv_bfloat16* src) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
 }
@@ -1016,6 +1004,146 @@ token_input_kernel(float* __restrict__ resid, int width, const __nv_bfloat16* __
   for (int i = 0; i < TI_CLUSTER; ++i) total += sums[i];
   const float inv = 1.0f / sqrtf(total / (float)width + eps);
   for (int n = n_lo + tid; n < n_hi; n += TI_THREADS) row[n] = x_s[n] + y_s[n - n_lo] * inv * norm_w[n];
+}
+
+// ---------------------------------------------------------------------------------------------
+// Embedding with a pair table: resid[t] = table[id_t] * scale + pairs[(id_(t-1) * mul_prev + id_t * mul_cur) mod buckets],
+// and row `buckets` of the pair table for a sequence's first token.  The token before a portion's first one is
+// the sequence's int32 state; the block of that first row reads it and then writes the portion's last
+// token there, so no other block touches it.  One block per row.
+template <typename T>
+__global__ void embed_pairs_kernel(const T* __restrict__ table, const T* __restrict__ pairs, long long mul_prev,
+                                   long long mul_cur, int buckets, float scale, const int* __restrict__ ids,
+                                   const int* __restrict__ fed, int num_fed, const int* __restrict__ positions,
+                                   int* __restrict__ last, float* __restrict__ resid, int width, int vocab,
+                                   const int* __restrict__ q_start, const int* __restrict__ q_len,
+                                   const int* __restrict__ seq_slots, int num_seqs, int* status) {
+  __shared__ int mine, before_s;
+  allow_dependents();
+  if (threadIdx.x == 0) mine = -1;
+  __syncthreads();
+  grid_dependency_wait();
+  const int t = blockIdx.x;
+  for (int s = threadIdx.x; s < num_seqs; s += blockDim.x)
+    if (q_start[s] == t && q_len[s] > 0) mine = s;
+  __syncthreads();
+  const int seq = mine;
+  const int id = token_of(ids, t, fed, num_fed, vocab);
+  if (threadIdx.x == 0) {
+    if (id < 0) atomicOr(status, VX_STATUS_BAD_TOKEN_ID);
+    int before = -1;
+    if (positions[t] > 0) before = seq >= 0 ? last[seq_slots[seq]] : t > 0 ? token_of(ids, t - 1, fed, num_fed, vocab) : -1;
+    if (seq >= 0) last[seq_slots[seq]] = max(0, token_of(ids, t + q_len[seq] - 1, fed, num_fed, vocab));
+    before_s = before;
+  }
+  __syncthreads();
+  const int before = before_s;
+  float* dst = resid + (size_t)t * width;
+  if (id < 0) {
+    for (int i = threadIdx.x; i < width; i += blockDim.x) dst[i] = 0.f;
+    return;
+  }
+  long long at = buckets;
+  if (before >= 0) {
+    at = ((long long)before * mul_prev + (long long)id * mul_cur) % buckets;
+    if (at < 0) at += buckets;
+  }
+  const T* a = table + (size_t)id * width;
+  const T* b = pairs + (size_t)at * width;
+  for (int i = threadIdx.x; i < width; i += blockDim.x) dst[i] = fmaf(to_float(a[i]), scale, to_float(b[i]));
+}
+
+// ---------------------------------------------------------------------------------------------
+// Queries and keys normed over the whole projection, then rotated.  A row holds q [H][D] | k [G][D] | v [G][D] (or q alone:
+// G = 0), every head padded with zeros to D; q_w [H * D] and k_w [G * D] are the norms' weights (0 in the
+// padding).  With rms over all of q (q_values of its columns are real) and over all of k:
+//     q <- rotate(q / rms * q_w) in place;   k_cache[slot] = rotate(k / rms * k_w);   v_cache[slot] = v
+// Rotation: dims i and i + rot / 2 (i < rot / 2) of a head turn by the tabulated angle of (position, i).
+// One block per row.
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(256)
+norm_rope_store_kernel(T* __restrict__ rows, long long stride, const int* __restrict__ positions,
+                       const float* __restrict__ cos_t, const float* __restrict__ sin_t, int max_pos,
+                       const float* __restrict__ q_w, const float* __restrict__ k_w, int q_values, int k_values, float eps,
+                       const int* __restrict__ slots, T* __restrict__ k_cache, T* __restrict__ v_cache,
+                       long long num_slots, int H, int G, int D, int rot, int* status) {
+  __shared__ float sums[2][8];
+  allow_dependents();
+  grid_dependency_wait();
+  constexpr int N = VEC ? Pack<T>::N : 1;
+  const int t = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, warps = blockDim.x >> 5;
+  T* row = rows + (size_t)t * stride;
+  const int q_cols = H * D, k_cols = G * D, half = rot >> 1;
+  auto load = [&](const T* p, float (&v)[N]) {
+    if constexpr (VEC) load_pack(p, v);
+    else v[0] = to_float(*p);
+  };
+  auto store = [&](T* p, const float (&v)[N]) {
+    if constexpr (VEC) store_pack(p, v);
+    else *p = from_float<T>(v[0]);
+  };
+  float sq = 0.f, sk = 0.f;
+  for (int i = tid * N; i < q_cols + k_cols; i += blockDim.x * N) {
+    float v[N], s = 0.f;
+    load(row + i, v);
+#pragma unroll
+    for (int e = 0; e < N; ++e) s = fmaf(v[e], v[e], s);
+    if (i < q_cols) sq += s;
+    else sk += s;
+  }
+  sq = warp_sum(sq);
+  sk = warp_sum(sk);
+  if (lane == 0) sums[0][warp] = sq, sums[1][warp] = sk;
+  __syncthreads();
+  sq = sk = 0.f;
+  for (int w = 0; w < warps; ++w) sq += sums[0][w], sk += sums[1][w];
+  const float q_inv = 1.0f / sqrtf(sq / (float)q_values + eps);
+  const float k_inv = G > 0 ? 1.0f / sqrtf(sk / (float)k_values + eps) : 0.f;
+  int pos = positions[t];
+  if (rot > 0 && (pos < 0 || pos >= max_pos)) {
+    if (tid == 0) atomicOr(status, VX_STATUS_BAD_POSITION);
+    pos = 0;
+  }
+  const int slot = G > 0 ? slots[t] : -1;
+  const bool slot_ok = slot >= 0 && (long long)slot < num_slots;
+  if (slot >= 0 && !slot_ok && tid == 0) atomicOr(status, VX_STATUS_BAD_SLOT);
+  const float* c = cos_t + (size_t)pos * half;
+  const float* s = sin_t + (size_t)pos * half;
+  // Packs of q and k (a pack of the low half with its partner; the high half's own turn passes), then of v.
+  const int per = D / N, total = (H + 2 * G) * per;
+  for (int idx = tid; idx < total; idx += blockDim.x) {
+    const int head = idx / per, d = (idx - head * per) * N;
+    const bool is_q = head < H, is_k = !is_q && head < H + G;
+    if (!is_q && !slot_ok) continue;
+    T* src = row + (size_t)head * D;
+    T* dst = is_q ? src : is_k ? k_cache + ((size_t)slot * G + head - H) * D : v_cache + ((size_t)slot * G + head - H - G) * D;
+    float v[N];
+    if (!is_q && !is_k) {
+      load(src + d, v);
+      store(dst + d, v);
+      continue;
+    }
+    const float inv = is_q ? q_inv : k_inv;
+    const float* w = is_q ? q_w + (size_t)head * D : k_w + (size_t)(head - H) * D;
+    if (d >= rot) {
+      load(src + d, v);
+#pragma unroll
+      for (int e = 0; e < N; ++e) v[e] *= inv * w[d + e];
+      store(dst + d, v);
+    } else if (d < half) {
+      float u[N];
+      load(src + d, v);
+      load(src + d + half, u);
+#pragma unroll
+      for (int e = 0; e < N; ++e) {
+        const float a = v[e] * inv * w[d + e], b = u[e] * inv * w[d + half + e];
+        v[e] = a * c[d + e] - b * s[d + e];
+        u[e] = b * c[d + e] + a * s[d + e];
+      }
+      store(dst + d, v);
+      store(dst + d + half, u);
+    }
+  }
 }
 
 }  // namespace vx
@@ -1201,27 +1329,46 @@ VX_API int vx_token_input(float* resid, int width, const void* w_gate, int dim, 
   }
   int lanes_log2 = 0;
   while (lanes_log2 < 5 && (8 << lanes_log2) < dim_pad) ++lanes_log2;
-  cudaLaunchConfig_t config = {};
-  config.gridDim = dim3(TI_CLUSTER, num_tokens);
-  config.blockDim = dim3(TI_THREADS);
-  config.dynamicSmemBytes = smem;
-  config.stream = stream;
-  static const bool serialised = [] {
-    const char* value = getenv("VELOX_B200_NO_PDL");
-    return value != nullptr && value[0] == '1';
-  }();
-  cudaLaunchAttribute attributes[2];
-  attributes[0].id = cudaLaunchAttributeClusterDimension;
-  attributes[0].val.clusterDim.x = TI_CLUSTER;
-  attributes[0].val.clusterDim.y = 1;
-  attributes[0].val.clusterDim.z = 1;
-  attributes[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-  attributes[1].val.programmaticStreamSerializationAllowed = 1;
-  config.attrs = attributes;
-  config.numAttrs = serialised ? 1 : 2;
-  return (int)cudaLaunchKernelEx(&config, token_input_kernel, resid, width, (const __nv_bfloat16*)w_gate, dim, dim_pad,
+  return (int)launch_pdl_cluster(token_input_kernel, dim3(TI_CLUSTER, num_tokens), dim3(TI_THREADS), smem, TI_CLUSTER,
+                                 stream, resid, width, (const __nv_bfloat16*)w_gate, dim, dim_pad,
                                  (const __nv_bfloat16*)table, table_stride, col, ids, fed, num_fed, vocab,
                                  (const __nv_bfloat16*)w_proj, norm_w, eps, lanes_log2, gate_rows, stage_gate, status);
+}
+
+VX_API int vx_embed_pairs(const void* table, const void* pairs, int dtype, long long mul_prev, long long mul_cur, int buckets,
+                          float scale, const int* ids, const int* fed, int num_fed, const int* positions, int* last,
+                          float* resid, int width, int vocab, const int* q_start, const int* q_len,
+                          const int* seq_slots, int num_seqs, int num_tokens, int* status, cudaStream_t stream) {
+  if (num_tokens <= 0) return 0;
+  if (buckets <= 0) return (int)cudaErrorInvalidValue;
+  const int threads = width >= 1024 ? 256 : 128;
+  VX_BY_DTYPE(dtype, launch_pdl(embed_pairs_kernel<T>, dim3(num_tokens), dim3(threads), 0, stream, (const T*)table,
+                                (const T*)pairs, mul_prev, mul_cur, buckets, scale, ids, fed, num_fed, positions, last,
+                                resid, width, vocab, q_start, q_len, seq_slots, num_seqs, status));
+  return (int)cudaGetLastError();
+}
+
+VX_API int vx_norm_rope_store(void* rows, int dtype, long long stride, const int* positions, const float* cos_t,
+                              const float* sin_t, int max_pos, const float* q_w, const float* k_w, int q_values,
+                              int k_values, float eps, const int* slots, void* k_cache, void* v_cache,
+                              long long num_slots, int num_tokens, int H, int G, int D, int rot, int* status,
+                              cudaStream_t stream) {
+  if (num_tokens <= 0) return 0;
+  if (H <= 0 || G < 0 || D <= 0 || rot < 0 || rot % 2 != 0 || rot > D || q_values <= 0 || (G > 0 && k_values <= 0))
+    return (int)cudaErrorInvalidValue;
+  const int pack = dtype == VX_DTYPE_F32 ? 4 : 8;
+  const bool vec = D % pack == 0 && (rot / 2) % pack == 0 && stride % pack == 0 && aligned16(rows) &&
+                   (G == 0 || (aligned16(k_cache) && aligned16(v_cache)));
+  const int work = (H + 2 * G) * D / (vec ? pack : 1);
+  const int threads = work >= 256 ? 256 : work > 64 ? 128 : 64;
+#define VX_NORM_ROPE(VEC)                                                                                              \
+  VX_BY_DTYPE(dtype, launch_pdl(norm_rope_store_kernel<T, VEC>, dim3(num_tokens), dim3(threads), 0, stream, (T*)rows, stride, \
+                                positions, cos_t, sin_t, max_pos, q_w, k_w, q_values, k_values, eps, slots, (T*)k_cache, \
+                                (T*)v_cache, num_slots, H, G, D, rot, status))
+  if (vec) { VX_NORM_ROPE(true) }
+  else { VX_NORM_ROPE(false) }
+#undef VX_NORM_ROPE
+  return (int)cudaGetLastError();
 }
 
 VX_TRACE_API(vx_heads)

@@ -5,7 +5,8 @@
 //                          a router's choice from its logits (or from the input, logits included, for
 //                          a few tokens): sigmoid scores, a correction per expert that only the choice
 //                          sees, the best groups of neighbouring experts, the `top` best experts of
-//                          those, their scores divided by their sum as weights
+//                          those, their scores divided by their sum as weights; or logits with a bias, the
+//                          `top` largest, their softmax as weights
 //   table_experts_kernel   one block per token: for each of the token's `top` experts act = the
 //                          activation of W_up[e] h and sum += weight * W_down[e] act, added to the
 //                          float32 residual stream.  (The plain form: any size.)
@@ -118,12 +119,21 @@ __device__ __forceinline__ float dot_row<__nv_bfloat16>(const __nv_bfloat16* __r
   return warp_sum(acc);
 }
 
+// A router's score of a logit: its sigmoid, chosen by score + correction, or (softmax) the logit with the
+// correction as a bias, which is then both.
+constexpr int ROUTER_SOFTMAX = 1;  // 0: sigmoid
+__device__ __forceinline__ void router_score(float z, float correction, int router, float* score, float* choice) {
+  const float v = router == ROUTER_SOFTMAX ? z + correction : 1.0f / (1.0f + expf(-z));
+  *score = v;
+  *choice = router == ROUTER_SOFTMAX ? v : v + correction;
+}
+
 // One warp: the choice of a token from its scores.  choice_s [experts] holds score + correction and is
 // used up, group_s [groups] is scratch.  A group's strength is the sum of its two best choice scores (of
 // its one, if it has one); experts outside the `keep` strongest groups cannot be chosen.  Ties go to the
 // lower number.
 __device__ __forceinline__ void choose_experts(float* choice_s, const float* score_s, float* group_s, int experts,
-                                               int groups, int keep, int top, float scale, int lane,
+                                               int groups, int keep, int top, float scale, int router, int lane,
                                                int* __restrict__ chosen, float* __restrict__ weights) {
   if (groups > 1) {
     const int size = experts / groups;
@@ -146,7 +156,7 @@ __device__ __forceinline__ void choose_experts(float* choice_s, const float* sco
     }
     __syncwarp();
   }
-  float sum = 0.f;
+  float sum = 0.f, largest = 0.f;
   for (int k = 0; k < top; ++k) {
     float best = -CUDART_INF_F;
     int at = experts;
@@ -161,21 +171,26 @@ __device__ __forceinline__ void choose_experts(float* choice_s, const float* sco
       if (other > best || (other == best && other_at < at)) { best = other; at = other_at; }
     }
     if (at >= experts) at = k;  // nothing comparable is left: still a valid expert
-    sum += score_s[at];
+    // The softmax over the chosen: against the largest logit, which comes first.
+    if (k == 0) largest = score_s[at];
+    sum += router == ROUTER_SOFTMAX ? expf(score_s[at] - largest) : score_s[at];
     if (lane == 0) {
       choice_s[at] = -CUDART_INF_F;
       chosen[k] = at;
     }
     __syncwarp();
   }
-  for (int k = lane; k < top; k += 32) weights[k] = score_s[chosen[k]] / (sum + 1e-20f) * scale;
+  for (int k = lane; k < top; k += 32) {
+    const float v = score_s[chosen[k]];
+    weights[k] = (router == ROUTER_SOFTMAX ? expf(v - largest) / sum : v / (sum + 1e-20f)) * scale;
+  }
 }
 
 constexpr int CE_WARPS = 4;
 
 __global__ void __launch_bounds__(CE_WARPS * 32)
 choose_experts_kernel(const float* __restrict__ logits, long long logit_stride, const float* __restrict__ correction,
-                      int experts, int groups, int keep, int top, float scale, int* __restrict__ chosen,
+                      int experts, int groups, int keep, int top, float scale, int router, int* __restrict__ chosen,
                       float* __restrict__ weights, int num_tokens) {
   extern __shared__ float ce_s[];  // per warp: choice scores [experts], scores [experts], groups [groups]
   allow_dependents();
@@ -185,13 +200,10 @@ choose_experts_kernel(const float* __restrict__ logits, long long logit_stride, 
   if (t >= num_tokens) return;
   float* choice_s = ce_s + (size_t)warp * (2 * experts + groups);
   float* score_s = choice_s + experts;
-  for (int i = lane; i < experts; i += 32) {
-    const float v = 1.0f / (1.0f + expf(-logits[(size_t)t * logit_stride + i]));
-    score_s[i] = v;
-    choice_s[i] = v + correction[i];
-  }
+  for (int i = lane; i < experts; i += 32)
+    router_score(logits[(size_t)t * logit_stride + i], correction[i], router, score_s + i, choice_s + i);
   __syncwarp();
-  choose_experts(choice_s, score_s, score_s + experts, experts, groups, keep, top, scale, lane, chosen + (size_t)t * top,
+  choose_experts(choice_s, score_s, score_s + experts, experts, groups, keep, top, scale, router, lane, chosen + (size_t)t * top,
                  weights + (size_t)t * top);
 }
 
@@ -202,7 +214,7 @@ __global__ void __launch_bounds__(512)
 route_rows_kernel(const T* __restrict__ h, long long h_stride, const float* __restrict__ resid,
                   const float* __restrict__ norm_w, float eps, T* __restrict__ h_out, const T* __restrict__ w_router, int width,
                   const float* __restrict__ correction, int experts, int groups, int keep, int top, float scale,
-                  int* __restrict__ chosen, float* __restrict__ weights) {
+                  int router, int* __restrict__ chosen, float* __restrict__ weights) {
   extern __shared__ __align__(16) float moe_s[];  // [width], choice [experts], scores [experts], groups [groups]
   float* choice_s = moe_s + (width + 3) / 4 * 4;
   float* score_s = choice_s + experts;
@@ -231,15 +243,11 @@ route_rows_kernel(const T* __restrict__ h, long long h_stride, const float* __re
   __syncthreads();
   for (int e = warp; e < experts; e += warps) {
     const float z = dot_row<T>(w_router + (size_t)e * width, moe_s, width, lane);
-    if (lane == 0) {
-      const float v = 1.0f / (1.0f + expf(-z));
-      score_s[e] = v;
-      choice_s[e] = v + correction[e];
-    }
+    if (lane == 0) router_score(z, correction[e], router, score_s + e, choice_s + e);
   }
   __syncthreads();
   if (warp == 0)
-    choose_experts(choice_s, score_s, score_s + experts, experts, groups, keep, top, scale, lane, chosen + (size_t)t * top,
+    choose_experts(choice_s, score_s, score_s + experts, experts, groups, keep, top, scale, router, lane, chosen + (size_t)t * top,
                    weights + (size_t)t * top);
 }
 
@@ -809,8 +817,8 @@ using namespace vx;
 // A router's choice: chosen int32 [tokens, top], weights float32 [tokens, top], from the logits float32
 // [tokens, logit_stride].
 VX_API int vx_choose_experts(const float* logits, long long logit_stride, const float* correction, int experts,
-                             int groups, int keep, int top, float scale, int* chosen, float* weights, int num_tokens,
-                             cudaStream_t stream) {
+                             int groups, int keep, int top, float scale, int router, int* chosen, float* weights,
+                             int num_tokens, cudaStream_t stream) {
   if (num_tokens <= 0) return 0;
   if (experts <= 0 || groups <= 0 || experts % groups != 0 || top <= 0 || keep <= 0 || keep > groups ||
       top > experts / groups * keep)
@@ -818,7 +826,7 @@ VX_API int vx_choose_experts(const float* logits, long long logit_stride, const 
   const size_t smem = sizeof(float) * CE_WARPS * (2 * (size_t)experts + groups);
   if (smem > 48 * 1024) return (int)cudaErrorInvalidValue;
   launch_pdl(choose_experts_kernel, dim3((num_tokens + CE_WARPS - 1) / CE_WARPS), dim3(CE_WARPS * 32), smem, stream, logits,
-             logit_stride, correction, experts, groups, keep, top, scale, chosen, weights, num_tokens);
+             logit_stride, correction, experts, groups, keep, top, scale, router, chosen, weights, num_tokens);
   return (int)cudaGetLastError();
 }
 
@@ -826,8 +834,8 @@ VX_API int vx_choose_experts(const float* logits, long long logit_stride, const 
 // h_out [tokens, width]; -1: sizes the kernel does not take.
 VX_API int vx_route_rows(const void* h, int dtype, long long h_stride, const float* resid, const float* norm_w, float eps,
                          void* h_out, const void* w_router, int width,
-                         const float* correction, int experts, int groups, int keep, int top, float scale, int* chosen,
-                         float* weights, int num_tokens, cudaStream_t stream) {
+                         const float* correction, int experts, int groups, int keep, int top, float scale, int router,
+                         int* chosen, float* weights, int num_tokens, cudaStream_t stream) {
   if (num_tokens <= 0) return 0;
   if (experts <= 0 || groups <= 0 || experts % groups != 0 || top <= 0 || keep <= 0 || keep > groups ||
       top > experts / groups * keep)
@@ -837,11 +845,12 @@ VX_API int vx_route_rows(const void* h, int dtype, long long h_stride, const flo
   const int threads = experts >= 16 ? 512 : (experts < 4 ? 128 : 32 * experts);
   if (dtype == VX_DTYPE_F32)
     launch_pdl(route_rows_kernel<float>, dim3(num_tokens), dim3(threads), smem, stream, (const float*)h, h_stride, resid,
-               norm_w, eps, (float*)h_out, (const float*)w_router, width, correction, experts, groups, keep, top, scale, chosen, weights);
+               norm_w, eps, (float*)h_out, (const float*)w_router, width, correction, experts, groups, keep, top, scale, router,
+               chosen, weights);
   else
     launch_pdl(route_rows_kernel<__nv_bfloat16>, dim3(num_tokens), dim3(threads), smem, stream, (const __nv_bfloat16*)h,
-               h_stride, resid, norm_w, eps, (__nv_bfloat16*)h_out, (const __nv_bfloat16*)w_router, width, correction, experts, groups, keep, top, scale, chosen,
-               weights);
+               h_stride, resid, norm_w, eps, (__nv_bfloat16*)h_out, (const __nv_bfloat16*)w_router, width, correction, experts, groups, keep, top, scale,
+               router, chosen, weights);
   return (int)cudaGetLastError();
 }
 

@@ -44,6 +44,10 @@ class CausalLM:
         self.final_norm = _build("norm", spec.final_norm, store, dtype, device)
         self.lm_head = _build("lm_head", spec.lm_head, store, dtype, device)
 
+        # A row per request that the embedding keeps (the token before), or None.
+        embedding_state = getattr(self.embedding, "state_needs", None)
+        self.embedding_needs = embedding_state() if embedding_state is not None else None
+
         positions: Dict[int, object] = {}
         self.blocks = []
         for layer in spec.layers:

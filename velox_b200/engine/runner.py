@@ -122,6 +122,8 @@ class StepContext:
     # int32 on the device, or None: the tokens the sampler drew in the step before, one per row.
     # A token id of -1 - r in this step's ids stands for row r of it (looked up by the embedding).
     fed_tokens: Optional[torch.Tensor] = None
+    # The embedding's state rows, one per slot (the last one for padding), or None.
+    embedding_state: Optional[torch.Tensor] = None
     # Which schedule entry is running (set by the model around every block).
     entry_index: int = 0
     # Columns of a part's first projection that belong to the block around it (a gate over the
@@ -280,6 +282,11 @@ class ModelRunner:
                         cache.page_size, max_num_seqs, self.dtype, self.device,
                     )
                 )
+        # The embedding's own row per state slot.
+        self.embedding_state: Optional[torch.Tensor] = None
+        if model.embedding_needs is not None:
+            needs = model.embedding_needs
+            self.embedding_state = torch.zeros((max_num_seqs + 1,) + tuple(needs.shape), dtype=needs.dtype, device=self.device)
         self._signatures = model.attention_signatures()
         # One counter per (merge item, KV head); the kernels leave them at zero.
         self._split_counters = torch.zeros(1 << 16, dtype=torch.int32, device=self.device)
@@ -325,6 +332,8 @@ class ModelRunner:
                 layer_cache.state[seq.slot].zero_()
             if layer_cache.block_state is not None:
                 layer_cache.block_state[seq.slot].zero_()
+        if self.embedding_state is not None:
+            self.embedding_state[seq.slot].zero_()
 
     def kv_cache_bytes(self) -> int:
         return sum(c.num_bytes() for c in self.layer_caches if not c.read_only)
@@ -641,6 +650,7 @@ class ModelRunner:
             workspace=self.workspace,
             plans=plans,
             fed_tokens=self.fed_tokens,
+            embedding_state=self.embedding_state,
             single_tokens=padded or (not round_shape and all(n == 1 for n in q_lens)),
             q_lens_host=[int(n) for n in q_len_arr],
             kv_lens_host=[int(n) for n in kv_len_arr],

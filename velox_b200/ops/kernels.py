@@ -8,6 +8,7 @@ functions raise.
 from __future__ import annotations
 
 import ctypes
+import math
 from typing import Optional
 
 import torch
@@ -191,11 +192,35 @@ def mixers():
         ]
         lib.vx_table_experts_runs.argtypes = lib.vx_table_experts_rows.argtypes
         lib.vx_choose_experts.argtypes = [
-            _ptr, _c_ll, _ptr, _c_int, _c_int, _c_int, _c_int, _c_f, _ptr, _ptr, _c_int, _ptr,
+            _ptr, _c_ll, _ptr, _c_int, _c_int, _c_int, _c_int, _c_f, _c_int, _ptr, _ptr, _c_int, _ptr,
         ]
         lib.vx_route_rows.argtypes = [
-            _ptr, _c_int, _c_ll, _ptr, _ptr, _c_f, _ptr, _ptr, _c_int, _ptr, _c_int, _c_int, _c_int, _c_int, _c_f, _ptr,
-            _ptr, _c_int, _ptr,
+            _ptr, _c_int, _c_ll, _ptr, _ptr, _c_f, _ptr, _ptr, _c_int, _ptr, _c_int, _c_int, _c_int, _c_int, _c_f, _c_int,
+            _ptr, _ptr, _c_int, _ptr,
+        ]
+        lib.vx_conv_act.argtypes = [
+            _ptr, _c_int, _c_ll, _c_int, _c_int, _ptr, _ptr, _ptr, _c_ll, _ptr, _c_ll, _ptr, _ptr, _ptr, _c_int, _c_int,
+            _c_int, _ptr,
+        ]
+        lib.vx_selective_max_state.restype = _c_int
+        lib.vx_selective_block_channels.argtypes = [_c_int]
+        lib.vx_selective_scan.argtypes = [
+            _ptr, _c_int, _c_ll, _ptr, _c_ll, _ptr, _ptr, _ptr, _c_ll, _ptr, _ptr, _c_ll, _ptr, _c_ll, _ptr, _c_ll, _c_int,
+            _c_int, _c_int, _ptr, _ptr, _ptr, _ptr, _ptr, _c_int, _c_int, _ptr,
+        ]
+        lib.vx_selective_step.argtypes = [
+            _ptr, _c_int, _c_ll, _ptr, _c_ll, _ptr, _c_int, _ptr, _ptr, _ptr, _ptr, _c_ll, _ptr, _c_ll, _ptr, _c_ll,
+            _c_int, _c_int, _ptr, _ptr, _c_int, _ptr,
+        ]
+        lib.vx_gated_linear_scratch.argtypes = [_c_int, _c_int, _c_int, _c_int]
+        lib.vx_gated_linear_scratch.restype = _c_ll
+        lib.vx_gated_linear_chunks.argtypes = [
+            _ptr, _ptr, _ptr, _c_int, _c_ll, _ptr, _c_ll, _ptr, _c_f, _c_f, _c_int, _c_int, _c_int, _ptr, _c_ll, _ptr, _c_ll,
+            _ptr, _c_ll, _ptr, _ptr, _ptr, _c_int, _c_int, _c_int, _ptr, _ptr,
+        ]
+        lib.vx_gated_linear_step.argtypes = [
+            _ptr, _ptr, _ptr, _c_int, _c_ll, _ptr, _c_ll, _ptr, _c_int, _ptr, _c_f, _c_f, _c_int, _c_int, _c_int, _ptr, _c_ll,
+            _ptr, _c_f, _ptr, _c_ll, _ptr, _c_ll, _ptr, _ptr, _c_int, _ptr,
         ]
         lib.vx_grouped_tile_rows.restype = _c_int
         lib.vx_table_experts_grouped.argtypes = [_ptr, _c_ll] + choice + [
@@ -241,6 +266,14 @@ def heads():
         lib.vx_token_input.argtypes = [
             _ptr, _c_int, _ptr, _c_int, _c_int, _ptr, _c_ll, _c_int, _ptr, _ptr, _c_int, _c_int, _ptr, _ptr, _c_f,
             _c_int, _ptr, _ptr,
+        ]
+        lib.vx_embed_pairs.argtypes = [
+            _ptr, _ptr, _c_int, _c_ll, _c_ll, _c_int, _c_f, _ptr, _ptr, _c_int, _ptr, _ptr, _ptr, _c_int, _c_int, _ptr, _ptr,
+            _ptr, _c_int, _c_int, _ptr, _ptr,
+        ]
+        lib.vx_norm_rope_store.argtypes = [
+            _ptr, _c_int, _c_ll, _ptr, _ptr, _ptr, _c_int, _ptr, _ptr, _c_int, _c_int, _c_f, _ptr, _ptr, _ptr, _c_ll, _c_int,
+            _c_int, _c_int, _c_int, _c_int, _ptr, _ptr,
         ]
         lib.vx_clamped_glu.argtypes = [_ptr, _c_int, _c_ll, _ptr, _c_ll, _c_int, _c_int, _c_f, _c_f, _c_f, _c_f, _ptr]
         _heads = lib
@@ -1778,6 +1811,144 @@ def gated_delta_step(x, b, a, per_channel, dt_bias, a_log, conv_weight_t, ring, 
     return True
 
 
+def conv_act(x, weight_t, bias, state, out, q_start, q_len, seq_slots, num_seqs, num_tokens, act) -> None:
+    """Causal convolution per channel with bias and activation over each sequence's tokens, rows in the compute
+    dtype, and the update of its state.  ``weight_t`` float32 [taps, channels], the current token's last; ``state``
+    float32 [slots, (taps - 1) * channels]: the last taps - 1 inputs of each slot's sequence, oldest first."""
+    for name, t in (("weight_t", weight_t), ("bias", bias)):
+        _need(t, torch.float32, name)
+    taps, channels = weight_t.shape
+    if x.shape[1] != channels or out.shape[1] != channels or bias.numel() != channels or out.dtype != x.dtype:
+        raise ValueError("conv_act: widths or dtypes do not agree")
+    if state.dtype != torch.float32 or (taps > 1 and state.shape[1] < (taps - 1) * channels):
+        raise ValueError("conv_act: the state is too small")
+    _check(mixers().vx_conv_act(_p(x), _code(x.dtype), _pitched(x, "x"), channels, taps, _p(weight_t), _p(bias), _p(state),
+                                state.stride(0), _p(out), _pitched(out, "out"), _p(q_start), _p(q_len), _p(seq_slots),
+                                num_seqs, num_tokens, act, _stream()), "conv_act")
+
+
+def _selective_check(x, dt_bias, a2, d_skip, z, out, state):
+    inner, states = a2.shape
+    for name, t in (("dt_bias", dt_bias), ("a2", a2), ("d_skip", d_skip)):
+        _need(t, torch.float32, name)
+    if x.shape[1] != inner or z.shape[1] != inner or out.shape[1] != inner or dt_bias.numel() != inner or d_skip.numel() != inner:
+        raise ValueError("selective scan: widths do not agree")
+    if z.dtype != x.dtype or out.dtype != x.dtype or state.dtype != torch.float32 or state.shape[1] < inner * states:
+        raise ValueError("selective scan: dtypes do not agree, or the state is too small")
+    return inner, states
+
+
+def selective_chunk(num_tokens: int, num_seqs: int, inner: int, states: int) -> int:
+    """Tokens of a chunk with which ``selective_scan`` should cut a step's portions (0: not at all): chunks run
+    side by side but make every decay twice, so they pay only where whole sequences leave SMs without work."""
+    blocks = -(-inner // int(mixers().vx_selective_block_channels(states))) * num_seqs
+    if num_tokens < 256 or 2 * blocks > 148:
+        return 0
+    # About two blocks an SM, in chunks of at least 64 tokens.
+    return max(64, -(-num_tokens * blocks // (2 * 148 * 16)) * 16)
+
+
+def selective_scan(x, dt, dt_bias, a2, bc, d_skip, z, out, state, q_start, q_len, seq_slots, num_seqs, num_tokens,
+                   chunk=0, chunk_states=None, chunk_dt=None) -> None:
+    """Per channel c and state n: ``S <- exp(dt A) S + dt x B``, ``out = (sum_n S C + D x) * silu(z)`` with ``dt =
+    softplus(dt + dt_bias)`` (``dt`` float32 logits) and ``a2 = A log2(e)`` float32 [inner, states]; ``bc`` rows hold B |
+    C; ``state`` float32 [slots, inner * states].  With ``chunk`` > 0 longer portions run in chunks of that many
+    tokens side by side, with float32 scratch ``chunk_states`` ((num_tokens // chunk + num_seqs + 1) * inner * states
+    values) and ``chunk_dt`` (as many times inner)."""
+    inner, states = _selective_check(x, dt_bias, a2, d_skip, z, out, state)
+    if dt.dtype != torch.float32 or dt.shape[1] != inner or bc.dtype != x.dtype or bc.shape[1] != 2 * states:
+        raise ValueError("selective_scan: dt or bc do not match")
+    if chunk > 0:
+        places = num_tokens // chunk + num_seqs + 1
+        _need(chunk_states, torch.float32, "chunk_states")
+        _need(chunk_dt, torch.float32, "chunk_dt")
+        if chunk_states.numel() < places * inner * states or chunk_dt.numel() < places * inner:
+            raise ValueError("selective_scan: the scratch is too small")
+    _check(mixers().vx_selective_scan(
+        _p(x), _code(x.dtype), _pitched(x, "x"), _p(dt), _pitched(dt, "dt"), _p(dt_bias), _p(a2), _p(bc), _pitched(bc, "bc"),
+        _p(d_skip), _p(z), _pitched(z, "z"), _p(out), _pitched(out, "out"), _p(state), state.stride(0), inner, states,
+        int(chunk), _p(chunk_states) if chunk > 0 else None, _p(chunk_dt) if chunk > 0 else None, _p(q_start), _p(q_len),
+        _p(seq_slots), num_seqs, num_tokens, _stream()), "selective_scan")
+
+
+def selective_step(x, low, w_dt, dt_bias, a2, d_skip, z, out, state, q_start, seq_slots, num_seqs) -> bool:
+    """One token of every sequence in one launch: ``selective_scan`` with ``dt = softplus(W_dt low + dt_bias)`` made
+    here from the first columns of the rows ``low | B | C``.  False: sizes the kernel does not take."""
+    inner, states = _selective_check(x, dt_bias, a2, d_skip, z, out, state)
+    rank = w_dt.shape[1]
+    _need(w_dt, x.dtype, "w_dt")
+    if w_dt.shape[0] != inner or low.dtype != x.dtype or low.shape[1] < rank + 2 * states:
+        raise ValueError("selective_step: low or w_dt do not match")
+    code = mixers().vx_selective_step(
+        _p(x), _code(x.dtype), _pitched(x, "x"), _p(low), _pitched(low, "low"), _p(w_dt), rank, _p(dt_bias), _p(a2),
+        _p(d_skip), _p(z), _pitched(z, "z"), _p(out), _pitched(out, "out"), _p(state), state.stride(0), inner, states,
+        _p(q_start), _p(seq_slots), num_seqs, _stream())
+    if code == -1:
+        return False
+    _check(code, "selective_step")
+    return True
+
+
+def _gated_linear_check(q, k, v, a_bias, state, heads, key_dim, value_dim) -> int:
+    stride = _pitched(q, "q")
+    if q.shape[1] != heads * key_dim or k.shape[1] != heads * key_dim or v.shape[1] != heads * value_dim:
+        raise ValueError("gated linear attention: widths do not match the heads")
+    if _pitched(k, "k") != stride or _pitched(v, "v") != stride or k.dtype != q.dtype or v.dtype != q.dtype:
+        raise ValueError("gated linear attention: q, k and v are columns of the same rows")
+    _need(a_bias, torch.float32, "a_bias")
+    if a_bias.numel() != heads * key_dim or state.dtype != torch.float32 or state.shape[1] < heads * key_dim * value_dim:
+        raise ValueError("gated linear attention: the bias or the state does not match the heads")
+    return stride
+
+
+def gated_linear_scratch(num_tokens: int, num_seqs: int, heads: int, key_dim: int) -> int:
+    """float32 values of scratch ``gated_linear_chunks`` wants; -1: a key size it does not take."""
+    return int(mixers().vx_gated_linear_scratch(num_tokens, num_seqs, heads, key_dim))
+
+
+def gated_linear_chunks(q, k, v, z, a_bias, q_scale, tau, heads, key_dim, value_dim, records, state, out, q_start, q_len,
+                        seq_slots, num_seqs, num_tokens, status) -> None:
+    """Gated linear attention over each sequence's tokens: per head ``S <- diag(alpha) S + k v^T``, ``out = S^T (q_scale
+    q)`` with ``alpha = sigmoid(z + a_bias)^(1 / tau)`` (``z`` float32 [tokens, heads * key_dim]); in chunks of 32 tokens
+    as small matrix products in float32.  ``records`` float32 scratch (``gated_linear_scratch``), ``state`` float32
+    [slots, heads * value_dim * key_dim], ``out`` float32 [tokens, heads * value_dim]."""
+    stride = _gated_linear_check(q, k, v, a_bias, state, heads, key_dim, value_dim)
+    _need(records, torch.float32, "records")
+    _need(status, torch.int32, "status")
+    if z.dtype != torch.float32 or z.shape[1] != heads * key_dim or out.dtype != torch.float32 or out.shape[1] != heads * value_dim:
+        raise ValueError("gated_linear_chunks: z or out do not match the heads")
+    _check(mixers().vx_gated_linear_chunks(
+        _p(q), _p(k), _p(v), _code(q.dtype), stride, _p(z), _pitched(z, "z"), _p(a_bias), float(q_scale),
+        math.log2(math.e) / float(tau), heads, key_dim, value_dim, _p(records), records.numel(), _p(state), state.stride(0),
+        _p(out), _pitched(out, "out"), _p(q_start), _p(q_len), _p(seq_slots), num_seqs, num_tokens, num_tokens, _p(status),
+        _stream()), "gated_linear_chunks")
+
+
+def gated_linear_step(q, k, v, low, a_up, a_bias, q_scale, tau, heads, key_dim, value_dim, gate, norm_weight, norm_eps,
+                      out, state, q_start, seq_slots, num_seqs) -> bool:
+    """One token of every sequence in one launch: the decay's logits ``a_up low`` (``low`` [tokens, rank], ``a_up``
+    [heads * key_dim, rank]), the state's update and read-out as in ``gated_linear_chunks``, every head's
+    read-out divided by its RMS, times ``norm_weight`` [value_dim], times ``silu(gate)``.  False: sizes the kernel
+    does not take."""
+    stride = _gated_linear_check(q, k, v, a_bias, state, heads, key_dim, value_dim)
+    _need(a_up, q.dtype, "a_up")
+    _need(norm_weight, torch.float32, "norm_weight")
+    rank = a_up.shape[1]
+    if a_up.shape[0] != heads * key_dim or low.dtype != q.dtype or low.shape[1] != rank or norm_weight.numel() != value_dim:
+        raise ValueError("gated_linear_step: the low-rank pair or the norm does not match the heads")
+    if gate.dtype != q.dtype or gate.shape[1] != heads * value_dim or out.dtype != q.dtype or out.shape[1] != heads * value_dim:
+        raise ValueError("gated_linear_step: gate or out do not match the heads")
+    code = mixers().vx_gated_linear_step(
+        _p(q), _p(k), _p(v), _code(q.dtype), stride, _p(low), _pitched(low, "low"), _p(a_up), rank, _p(a_bias),
+        float(q_scale), math.log2(math.e) / float(tau), heads, key_dim, value_dim, _p(gate), _pitched(gate, "gate"),
+        _p(norm_weight), float(norm_eps), _p(out), _pitched(out, "out"), _p(state), state.stride(0), _p(q_start),
+        _p(seq_slots), num_seqs, _stream())
+    if code == -1:
+        return False
+    _check(code, "gated_linear_step")
+    return True
+
+
 def dual_norm_mean(a, b, w_a, w_b, eps, scale, num_tokens, resid=None, out=None) -> None:
     """scale * (rms_norm(a) * w_a + rms_norm(b) * w_b): added to ``resid`` (float32) or written
     to ``out``."""
@@ -1855,11 +2026,17 @@ def _expert_sizes(w_up, form):
     return experts, (rows // 2 if form.gated else rows), width
 
 
-def choose_experts(logits, correction, groups, keep, top, scale, chosen, weights, num_tokens) -> None:
+# How a router scores: sigmoids with a correction that only the choice sees, or logits with the correction as a
+# bias whose softmax over the chosen experts gives the weights.
+ROUTER_SIGMOID, ROUTER_SOFTMAX = 0, 1
+
+
+def choose_experts(logits, correction, groups, keep, top, scale, chosen, weights, num_tokens, router=ROUTER_SIGMOID) -> None:
     """A router's choice from its float32 logits [tokens, experts]: scores sigmoid(logit); the ``top`` largest
     score + correction among the ``keep`` strongest of ``groups`` groups of neighbours (a group's strength:
     its two largest score + correction), their numbers into ``chosen`` int32 [tokens, top] and their scores
-    over the scores' sum (+ 1e-20), times ``scale``, into ``weights`` float32 [tokens, top]."""
+    over the scores' sum (+ 1e-20), times ``scale``, into ``weights`` float32 [tokens, top].  With ``router``
+    ``ROUTER_SOFTMAX`` the score is logit + correction and the weights are the softmax over the chosen scores."""
     _need(correction, torch.float32, "correction")
     _need(chosen, torch.int32, "chosen")
     _need(weights, torch.float32, "weights")
@@ -1868,11 +2045,13 @@ def choose_experts(logits, correction, groups, keep, top, scale, chosen, weights
     if chosen.numel() < num_tokens * top or weights.numel() < num_tokens * top:
         raise ValueError("choose_experts: the outputs do not hold the tokens")
     _check(mixers().vx_choose_experts(_p(logits), _pitched(logits, "logits"), _p(correction), correction.numel(), groups,
-                                      keep, top, float(scale), _p(chosen), _p(weights), num_tokens, _stream()),
+                                      keep, top, float(scale), int(router), _p(chosen), _p(weights), num_tokens,
+                                      _stream()),
            "choose_experts")
 
 
-def route_rows(h, w_router, correction, groups, keep, top, scale, chosen, weights, num_tokens, norm=None) -> bool:
+def route_rows(h, w_router, correction, groups, keep, top, scale, chosen, weights, num_tokens, norm=None,
+               router=ROUTER_SIGMOID) -> bool:
     """``choose_experts`` with the logits ``w_router h`` made in the same launch, a block per token (few
     tokens, and the float32 path).  ``norm`` = (resid, weight, eps): h is made here, ``resid / rms(resid) *
     weight``, and written to ``h``.  False: a row does not fit a block's shared memory."""
@@ -1894,7 +2073,8 @@ def route_rows(h, w_router, correction, groups, keep, top, scale, chosen, weight
         raise ValueError("route_rows: the outputs do not hold the tokens")
     code = mixers().vx_route_rows(_p(h), _code(h.dtype), _pitched(h, "h"), _p(resid), _p(norm_weight), float(eps),
                                   _p(h) if resid is not None else None, _p(w_router), width, _p(correction), experts,
-                                  groups, keep, top, float(scale), _p(chosen), _p(weights), num_tokens, _stream())
+                                  groups, keep, top, float(scale), int(router), _p(chosen), _p(weights), num_tokens,
+                                  _stream())
     if code == -1:
         return False
     _check(code, "route_rows")
@@ -2206,3 +2386,48 @@ def token_input(resid, w_gate, dim, table, col, ids, fed, w_proj, norm_weight, e
         return False
     _check(code, "token_input")
     return True
+
+
+def embed_pairs(table, pairs, mul_prev, mul_cur, scale, ids, fed, positions, last, resid, q_start, q_len, seq_slots,
+                num_seqs, num_tokens, status) -> None:
+    """``resid[t] = table[id_t] * scale + pairs[(id_(t-1) * mul_prev + id_t * mul_cur) mod buckets]``, the pair table's
+    last row (number ``buckets``) for a sequence's first token.  ``last`` int32, one per state slot: the sequence's
+    token before this step, read and rewritten.  Ids of ``-1 - r`` stand for row r of ``fed``."""
+    _need(ids, torch.int32, "ids")
+    _need(last, torch.int32, "last")
+    _need(resid, torch.float32, "resid")
+    _need(table, table.dtype, "table")
+    _need(pairs, table.dtype, "pairs")
+    vocab, width = table.shape
+    if pairs.shape[1] != width or resid.shape[1] != width or resid.shape[0] < num_tokens or ids.numel() < num_tokens:
+        raise ValueError("embed_pairs: sizes do not agree")
+    _check(heads().vx_embed_pairs(_p(table), _p(pairs), _code(table.dtype), int(mul_prev), int(mul_cur), pairs.shape[0] - 1,
+                                  float(scale), _p(ids), _p(fed), 0 if fed is None else fed.numel(), _p(positions),
+                                  _p(last), _p(resid), width, vocab, _p(q_start), _p(q_len), _p(seq_slots), num_seqs,
+                                  num_tokens, _p(status), _stream()), "embed_pairs")
+
+
+def norm_rope_store(rows, positions, cos, sin, rotary_dim, q_weight, k_weight, q_values, k_values, eps, slots, k_cache,
+                    v_cache, num_tokens, num_heads, num_kv_heads, head_dim, status) -> None:
+    """Rows q | k | v (``num_kv_heads`` 0: q alone) with every head padded to ``head_dim``: q and k each divided by
+    the RMS over its whole projection (``q_values`` / ``k_values`` real columns), times a weight per column, rotated
+    (dims i and i + rotary_dim / 2 of a head), q in place, k and v into the cache at ``slots``."""
+    _need(q_weight, torch.float32, "q_weight")
+    if q_weight.numel() != num_heads * head_dim or rows.shape[1] < (num_heads + 2 * num_kv_heads) * head_dim:
+        raise ValueError("norm_rope_store: the rows or the query norm do not match the heads")
+    num_slots = 0
+    if num_kv_heads:
+        _need(k_weight, torch.float32, "k_weight")
+        _need(k_cache, rows.dtype, "k_cache")
+        _need(v_cache, rows.dtype, "v_cache")
+        if k_weight.numel() != num_kv_heads * head_dim or k_cache.shape[2:] != (num_kv_heads, head_dim):
+            raise ValueError("norm_rope_store: the key norm or the cache do not match the heads")
+        num_slots = k_cache.shape[0] * k_cache.shape[1]
+    if rotary_dim > 0 and (cos.dtype != torch.float32 or cos.shape[1] != rotary_dim // 2):
+        raise ValueError("norm_rope_store: cos/sin tables do not match the rotary width")
+    _check(heads().vx_norm_rope_store(
+        _p(rows), _code(rows.dtype), _pitched(rows, "rows"), _p(positions), _p(cos) if rotary_dim else None,
+        _p(sin) if rotary_dim else None, cos.shape[0] if rotary_dim else 0, _p(q_weight),
+        _p(k_weight) if num_kv_heads else None, int(q_values), int(k_values), float(eps), _p(slots),
+        _p(k_cache) if num_kv_heads else None, _p(v_cache) if num_kv_heads else None, num_slots, num_tokens, num_heads,
+        num_kv_heads, head_dim, int(rotary_dim), _p(status), _stream()), "norm_rope_store")

@@ -16,6 +16,12 @@ q | k | v in the one projection); ``values_from_keys``: there is no value projec
 values are its keys as projected (bias included), before the rotation.  Such a part takes its
 matrices as ``q.weight``, ``k.weight``, ``v.weight`` (and biases) instead of one ``qkv.weight``.
 
+``qk_norm`` (an eps; weights ``q_norm``, ``k_norm`` of the projections' sizes): q and k are each divided by the RMS over
+their whole projection, all heads together, and multiplied by a weight per column before the rotation; norm,
+rotation and the cache's writes are then one kernel.  ``keys_from_cache``: the part has no key and value
+projections; it reads the keys and values that another schedule entry has cached (the entry's cache is
+``read_only``).
+
 Changes to the scores, made inside the attention kernels: ``distance_bias`` (weights ``bias_r1``,
 ``bias_r2``, one number each per query head): ``r1 ln(1 + r2 (i - j))`` is taken off the score of
 query i and key j; ``sink_zero``: one more term of score 0 and no value in every softmax
@@ -32,7 +38,7 @@ import torch
 
 from ..ops import kernels
 from ..ops.linear import linear, qkv_rope_linear, use_tensor_core_kernel
-from .base import CacheNeeds, Mixer, PagedCacheSpec
+from .base import CacheNeeds, Mixer, PagedCacheSpec, product_of
 from .registry import register_part
 
 # VELOX_B200_NO_ROPE_FUSION=1 always rotates in a kernel of its own (for bisecting).
@@ -77,6 +83,8 @@ class Attention(Mixer):
         self.b_qkv = None
         self.b_qkv_lowp = None
         self.values_from_keys = False
+        self.key_dim = self.value_dim = self.head_dim
+        self.own_keys = not params.get("keys_from_cache", False)
         if "qkv.weight" in weights:
             self.proj_width = self.qkv_width
             self.w_qkv = self.expect("qkv.weight", (self.qkv_width, self.hidden_size))
@@ -85,6 +93,12 @@ class Attention(Mixer):
             self.w_out = self.expect("out.weight", (self.hidden_size, self.q_size))
         else:
             self._fuse_padded(params, dtype, device)
+        self.qk_eps = params.get("qk_norm")
+        if self.qk_eps is None:
+            if not self.own_keys:
+                raise ValueError("attention: keys_from_cache goes with qk_norm")
+        else:
+            self._build_qk_norm()
         if self.b_qkv is not None and dtype != torch.float32:
             self.b_qkv_lowp = self.b_qkv.to(dtype)
         # Compile (or find) the kernels for this head size now, not in the first step.
@@ -101,6 +115,10 @@ class Attention(Mixer):
         if not (0 < kd <= D and 0 < vd <= D):
             raise ValueError(f"key_dim={kd} and value_dim={vd} must lie within head_dim={D}")
         self.key_dim, self.value_dim = kd, vd
+        if not self.own_keys:
+            if self.head_gate or params.get("values_from_keys", False):
+                raise ValueError("keys_from_cache goes with neither a gate per head nor values_from_keys")
+            self.qkv_width = self.q_size
 
         def padded_heads(t, heads, size):
             t = t.reshape(heads, size, *t.shape[1:])
@@ -121,15 +139,17 @@ class Attention(Mixer):
                     self.position, "layout", None) != "half":
                 raise ValueError("values_from_keys goes with the rotary_half position part and no gate per head")
             self.qkv_width = self.q_size + self.kv_size
-        pieces = [padded_heads(self.expect("q.weight", (H * kd, E)), H, kd),
-                  padded_heads(self.expect("k.weight", (G * kd, E)), G, kd)]
-        if not from_keys:
+        pieces = [padded_heads(self.expect("q.weight", (H * kd, E)), H, kd)]
+        if self.own_keys:
+            pieces.append(padded_heads(self.expect("k.weight", (G * kd, E)), G, kd))
+        if self.own_keys and not from_keys:
             pieces.append(padded_heads(self.expect("v.weight", (G * vd, E)), G, vd))
         bias = None
         if params.get("qkv_bias", False):
-            bias = [padded_heads(self.expect("q.bias", (H * kd,)), H, kd),
-                    padded_heads(self.expect("k.bias", (G * kd,)), G, kd)]
-            if not from_keys:
+            bias = [padded_heads(self.expect("q.bias", (H * kd,)), H, kd)]
+            if self.own_keys:
+                bias.append(padded_heads(self.expect("k.bias", (G * kd,)), G, kd))
+            if self.own_keys and not from_keys:
                 bias.append(padded_heads(self.expect("v.bias", (G * vd,)), G, vd))
         if self.head_gate:
             pieces.append(self.expect("gate.weight", (H, E)))
@@ -152,6 +172,23 @@ class Attention(Mixer):
         self.w_out = w_out
         for name in ("q.weight", "k.weight", "v.weight", "q.bias", "k.bias", "v.bias", "gate.weight"):
             self.weights.pop(name, None)
+
+    def _build_qk_norm(self) -> None:
+        """The norms' weights spread over the padded heads (0 in the padding)."""
+        if self.head_gate or self.values_from_keys or not hasattr(self.position, "rotate_and_store") or getattr(
+                self.position, "layout", "half") != "half":
+            raise ValueError("qk_norm goes with rotary_half or no positions, and with neither a gate per head nor "
+                             "values_from_keys")
+
+        def spread(name, heads):
+            t = self.expect(name, (heads * self.key_dim,)).to(torch.float32).reshape(heads, self.key_dim)
+            out = t.new_zeros(heads, self.head_dim)
+            out[:, : self.key_dim] = t
+            return out.reshape(-1).contiguous()
+
+        self.q_norm = spread("q_norm", self.num_heads)
+        self.k_norm = spread("k_norm", self.num_kv_heads) if self.own_keys else None
+        kernels.heads()
 
     def cache_needs(self) -> CacheNeeds:
         return CacheNeeds(paged=PagedCacheSpec(self.num_kv_heads, self.head_dim, self.window,
@@ -176,6 +213,17 @@ class Attention(Mixer):
         # Projection, rotation and cache write in one kernel, where the position encoding
         # offers its tables and the kernel takes the shape (it says no otherwise).
         tables = None
+        if not self.own_keys and not cache.read_only:
+            raise ValueError("an attention part without keys of its own needs another entry's cache")
+        if self.qk_eps is not None:
+            linear(x, self.w_qkv, self.b_qkv, qkv, T, self.b_qkv_lowp, status=ctx.status)
+            store = self.own_keys and k_cache is not None
+            kernels.norm_rope_store(
+                qkv, ctx.positions, getattr(self.position, "cos", None), getattr(self.position, "sin", None),
+                getattr(self.position, "rotary_dim", 0), self.q_norm, self.k_norm, self.num_heads * self.key_dim,
+                self.num_kv_heads * self.key_dim, self.qk_eps, group.slot_mapping, k_cache, v_cache, T, self.num_heads,
+                self.num_kv_heads if store else 0, self.head_dim, ctx.status)
+            return self._attend(qkv, ctx, cache, group, T)
         if _FUSE_ROPE and not self.values_from_keys:
             tables = getattr(self.position, "full_rotation_tables", lambda: None)()
         if tables is None or not qkv_rope_linear(
@@ -188,7 +236,10 @@ class Attention(Mixer):
             else:
                 self.position.rotate_and_store(qkv, ctx, group.slot_mapping, k_cache, v_cache,
                                                self.num_heads, self.num_kv_heads)
+        return self._attend(qkv, ctx, cache, group, T)
 
+    def _attend(self, qkv, ctx, cache, group, T):
+        ws = ctx.workspace
         attn = ws.get(f"attention.out{self.q_size}", (ws.max_tokens, self.q_size), self.dtype)
         plan = ctx.attention_plan(cache.group, self.attention_signature())
         for kind, items, count in plan.launches:
@@ -223,6 +274,4 @@ class Attention(Mixer):
             if mirror is not None:
                 ctx.residual_mirror_written = True
             return None
-        out = ws.get("mixer.out", (ws.max_tokens, self.hidden_size), self.dtype)
-        linear(attn, self.w_out, None, out, T, status=ctx.status)
-        return out
+        return product_of(attn, self.w_out, ctx, T)

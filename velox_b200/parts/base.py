@@ -35,7 +35,8 @@ stream, set by the block around the calls) itself.
 ``Block.forward(hidden, ctx, cache)``: the arrangement of norms, mixer and feed-forward around
     the residual stream; ``hidden`` carries (resid, pending delta).
 
-``Embedding.forward(ids, resid, ctx)``, ``LMHead.forward(x, num_rows, ctx) -> float32 [R, V]``.
+``Embedding.forward(ids, resid, ctx)``; ``Embedding.state_needs()`` may declare a ``StateSpec``, a row per request
+    that it finds as ``ctx.embedding_state``.  ``LMHead.forward(x, num_rows, ctx) -> float32 [R, V]``.
 """
 from __future__ import annotations
 
@@ -124,10 +125,27 @@ class PendingSums:
     """A part's product as float32 rows into which its last projection has added its shares (K cut
     into chunks of independent CTAs): what a block may get from a part instead of a tensor in the
     compute dtype.  ``bias`` (float32, or None) still has to be added.  The buffer was zero before
-    the projection and whoever reads the rows sets them to zero again."""
+    the projection and whoever reads the rows sets them to zero again.  Parts that have no buffer of
+    their own share ``block.sums``."""
 
     sums: torch.Tensor
     bias: Optional[torch.Tensor] = None
+
+
+def product_of(x, weight, ctx, num_rows: int, name: str = "mixer.out"):
+    """A mixer's last product ``x @ weight.T`` for a block that joins it itself: rows in the compute dtype, or,
+    for small steps and a block that takes them, float32 sums (``PendingSums``), K cut into chunks whose
+    CTAs need not wait for one another."""
+    from ..ops.linear import linear, use_tensor_core_kernel
+
+    ws = ctx.workspace
+    if ctx.takes_pending_sums and ctx.status is not None and use_tensor_core_kernel(x, weight, num_rows):
+        sums = ws.get("block.sums", (ws.max_tokens, weight.shape[0]), torch.float32)
+        linear(x, weight, None, sums, num_rows, status=ctx.status, accumulate=True)
+        return PendingSums(sums)
+    out = ws.get(name, (ws.max_tokens, weight.shape[0]), x.dtype)
+    linear(x, weight, None, out, num_rows, status=ctx.status)
+    return out
 
 
 class Part:

@@ -175,18 +175,19 @@ class PostNormBlock:
         source = x_in if lowp is None else lowp
 
         ctx.residual = None
+        ctx.residual_scale = None
         ctx.side_output = None
+        ctx.takes_pending_sums = True
         mixed = self.mixer.forward(source, ctx, cache)
         last = self.feed_forward is None
         self._join(x_in, work, mixed, ctx.side_output, self.norm_mixer, T, lowp, store, mix_out, last)
         if not last:
             source = work if lowp is None else lowp
             ctx.side_output = None
-            ctx.takes_pending_sums = lowp is not None
             product = self.feed_forward.forward(source, ctx)
-            ctx.takes_pending_sums = False
             self._join(work, work, product, ctx.side_output, self.norm_feed_forward, T, lowp, store, mix_out, True)
         ctx.side_output = None
+        ctx.takes_pending_sums = False
         hidden.resid = mix_out if self.depth_mix else work
         hidden.delta = None
         hidden.lowp = lowp
@@ -200,7 +201,7 @@ class PostNormBlock:
             resid_in, resid_out, delta, gate, norm.weight, norm.eps, norm.center, num_rows, lowp_out=lowp,
             history=store if mixing else None, mix_weights=self.mix_weight if mixing else None,
             mix_out=mix_out if mixing else None, sums=sums, sums_bias=bias,
-            compute_dtype=None if sums is None else lowp.dtype,
+            compute_dtype=None if sums is None else self.mixer.dtype,
         )
 
 

@@ -6,13 +6,17 @@ import torch
 
 from ..ops import kernels
 from ..ops.linear import linear, use_tensor_core_kernel
-from .base import Part
+from .base import Part, StateSpec
 from .registry import register_part
 
 
 @register_part("embedding", "token_embedding")
 class TokenEmbedding(Part):
-    """``resid[t] = table[ids[t]] * scale``, widened to the float32 residual stream (``scale``: 1)."""
+    """``resid[t] = table[ids[t]] * scale``, widened to the float32 residual stream (``scale``: 1).
+
+    ``bigram`` ({buckets, mul_prev, mul_cur}; weight ``bigram`` [buckets + 1, width]): row ``(previous token * mul_prev +
+    token * mul_cur) mod buckets`` of a second table is added, its last row for a sequence's first token.  The
+    previous token of a request is a state row of the embedding (int32)."""
 
     def __init__(self, params, weights, dtype, device) -> None:
         super().__init__(params, weights, dtype, device)
@@ -20,8 +24,22 @@ class TokenEmbedding(Part):
         self.hidden_size = int(params["hidden_size"])
         self.scale = float(params.get("scale", 1.0))
         self.table = self.expect("weight", (self.vocab_size, self.hidden_size))
+        self.pairs = None
+        if params.get("bigram"):
+            b = params["bigram"]
+            self.mul_prev, self.mul_cur = int(b["mul_prev"]), int(b["mul_cur"])
+            self.pairs = self.expect("bigram", (int(b["buckets"]) + 1, self.hidden_size))
+            kernels.heads()
+
+    def state_needs(self):
+        return None if self.pairs is None else StateSpec((1,), torch.int32)
 
     def forward(self, ids, resid, ctx) -> None:
+        if self.pairs is not None:
+            kernels.embed_pairs(self.table, self.pairs, self.mul_prev, self.mul_cur, self.scale, ids,
+                                getattr(ctx, "fed_tokens", None), ctx.positions, ctx.embedding_state, resid, ctx.q_start,
+                                ctx.q_len, ctx.seq_slots, ctx.num_seqs, ctx.num_tokens, ctx.status)
+            return
         # ctx.fed_tokens: the sampler's tokens of the step before, for ids that name one of them.
         kernels.embed(self.table, ids[: ctx.num_tokens], resid, ctx.status, getattr(ctx, "fed_tokens", None),
                       self.scale)

@@ -395,11 +395,15 @@ class RoutedExperts(FeedForward):
         largest c;   the ``top`` experts of those with the largest c
         out = scale * sum_e s_e / (sum of the chosen s + 1e-20) * expert_e(h)
 
+    or, with ``router`` "softmax" (no groups): logits ``z = W_router h + correction``, the ``top`` experts with the
+    largest z, weighted by the softmax over the chosen z (times ``scale``).
+
     ``router.weight`` [experts, width], ``router.correction`` [experts]; ``gate_up.weight`` holds, expert after
     expert, the gate rows and the up rows; ``down.weight`` the experts' down matrices.  ``shared``:
     parameters of a ``clamped_glu`` part that runs for every token beside them (weights with the prefix
     ``shared.``).  The router's logits, scores and weights are float32; the part adds its result into
-    the float32 stream itself, times the block's factors where it has them."""
+    the float32 stream itself, times the block's factors where it has them, or hands over float32 sums
+    to a block that takes them."""
 
     takes_padded_steps = True
     takes_residual_scale = True
@@ -414,6 +418,11 @@ class RoutedExperts(FeedForward):
         self.groups = int(params.get("groups", 1))
         self.keep = int(params.get("keep", self.groups))
         self.router_scale = float(params.get("router_scale", 1.0))
+        if params.get("router", "sigmoid") not in ("sigmoid", "softmax"):
+            raise ValueError(f"routed_experts: router is 'sigmoid' or 'softmax', not {params.get('router')!r}")
+        self.router = kernels.ROUTER_SOFTMAX if params.get("router") == "softmax" else kernels.ROUTER_SIGMOID
+        if self.router == kernels.ROUTER_SOFTMAX and self.groups != 1:
+            raise ValueError("routed_experts: a softmax router has no groups")
         self.form = dict(gated=True, limit=float(params.get("limit") or 0.0), alpha=float(params.get("alpha", 1.0)),
                          up_shift=float(params.get("up_shift", 0.0)), cubic=float(params.get("cubic", 0.0)))
         if X % self.groups or not 0 < self.keep <= self.groups:
@@ -457,14 +466,14 @@ class RoutedExperts(FeedForward):
             rows = x.out if pending is not None else x.materialize() if hasattr(x, "materialize") else x
             norm = None if pending is None else (pending.resid, pending.weight, pending.eps)
             if kernels.route_rows(rows, self.w_router, self.correction, self.groups, self.keep, self.top,
-                                  self.router_scale, chosen, weights, T, norm=norm):
+                                  self.router_scale, chosen, weights, T, norm=norm, router=self.router):
                 return rows, chosen, weights
         if hasattr(x, "materialize"):
             x = x.materialize()
         logits = ws.get(f"routed_experts.logits{self.experts}", (ws.max_tokens, self.experts), torch.float32)
         linear(x, self.w_router, None, logits, T, status=ctx.status)
         kernels.choose_experts(logits, self.correction, self.groups, self.keep, self.top, self.router_scale, chosen,
-                               weights, T)
+                               weights, T, router=self.router)
         return x, chosen, weights
 
     def _experts(self, x, chosen, weights, ctx, target, scale, T) -> None:
@@ -499,7 +508,10 @@ class RoutedExperts(FeedForward):
         ws = ctx.workspace
         stream, scale = ctx.residual, ctx.residual_scale
         target = stream
-        if target is None:
+        pending = target is None and ctx.takes_pending_sums
+        if pending:
+            target = ws.get("block.sums", (ws.max_tokens, self.hidden_size), torch.float32)
+        elif target is None:
             target = ws.get(f"routed_experts.sums{self.hidden_size}", (ws.max_tokens, self.hidden_size), torch.float32)
             target[:T].zero_()
         x, chosen, weights = self._route(x, ctx, T)
@@ -512,4 +524,6 @@ class RoutedExperts(FeedForward):
                 kernels.join_norm(target, product, None, T, scale=scale)
         if stream is not None:
             return None
+        if pending:
+            return PendingSums(target)
         return _lowered(target, ws, self.dtype, T, "routed_experts.out")

@@ -15,7 +15,9 @@ class RMSNorm(Norm):
     ``weight_offset`` c: the stored weight lies around zero and the factor is ``c + weight``
     (added once, in float32, when the part is built).  ``scalar_weight``: the stored weight is one
     number for all coordinates (a tensor without dimensions), spread over the row when the part
-    is built, so every kernel that takes a norm's weight vector takes this norm too."""
+    is built, so every kernel that takes a norm's weight vector takes this norm too.  ``weight_scale``: a
+    constant factor on the norm's output, multiplied into the weight when the part is built (a
+    sublayer's share of the stream, where the norm sits on the sublayer's result)."""
 
     def __init__(self, params, weights, dtype, device) -> None:
         super().__init__(params, weights, dtype, device)
@@ -28,6 +30,9 @@ class RMSNorm(Norm):
         offset = float(params.get("weight_offset", 0.0))
         if offset != 0.0:
             self.weight = (self.weight.to(torch.float32) + offset).contiguous()
+        scale = float(params.get("weight_scale", 1.0))
+        if scale != 1.0:
+            self.weight = (self.weight.to(torch.float32) * scale).contiguous()
 
     def forward(self, resid, delta, out, num_rows, rows=None, write_resid=True):
         if isinstance(delta, PendingJoin):

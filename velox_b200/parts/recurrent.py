@@ -39,17 +39,30 @@ q``, divided by its root mean square, times a weight shared by the heads, times 
 ``sigmoid``), then W_o.  The decay's logits and the gate's come from the layer's input directly or
 through a low-rank pair.  (State: S and a ring of the convolution's last inputs.)
 
+``selective_scan``: one projection of the input gives ``x | z`` (``inner`` channels each); x passes a causal convolution
+per channel with a bias and SiLU; a second product of x gives ``low | B | C`` (``rank``, ``state_size``, ``state_size``) and a
+third, of low, the step sizes' logits, ``dt = softplus(W_dt low + bias)`` per channel; with ``A = -exp(A_log)`` the
+state of channel c goes ``S[c, n] <- exp(dt_c A[c, n]) S[c, n] + dt_c x_c B_n`` and the result is ``W_o ((sum_n S[c, n] C_n +
+D_c x_c) * silu(z_c))``.  (Gu and Dao, "Mamba: Linear-Time Sequence Modeling with Selective State Spaces".)
+
+``gated_linear_attention``: ``S <- diag(alpha) S + k v^T`` per head (``dim`` x ``value_dim``, float32) with ``alpha =
+sigmoid(W_up (W_low x) + bias)^(1 / tau)`` per key channel, read by ``S^T (dim^(-1/2) q)``; every head's result is
+divided by its root mean square, times a weight shared by the heads, times ``silu(W_g x)``, then W_o.  (Yang et al.,
+"Gated Linear Attention Transformers with Hardware-Efficient Training".)
+
 ``side_by_side``: two mixers read the same input; the result is ``scale * (rms_norm(left) * w_l
 + rms_norm(right) * w_r)`` over the model width, or, with ``join`` = "weighted_sum",
 ``left_scale * left + right_scale * right`` without norms.
 """
 from __future__ import annotations
 
+import math
+
 import torch
 
 from ..ops import kernels
-from ..ops.linear import linear, use_tensor_core_kernel
-from .base import CacheNeeds, Mixer, StateSpec
+from ..ops.linear import SMALL_STEP_TOKENS, linear, use_tensor_core_kernel
+from .base import CacheNeeds, Mixer, StateSpec, product_of
 from .registry import part_class, register_part
 
 _ACTS = {"none": kernels.ACT_NONE, "silu": kernels.ACT_SILU, "gelu_tanh": kernels.ACT_GELU_TANH,
@@ -69,6 +82,15 @@ def _pad_rows(weight: torch.Tensor, multiple: int = 8) -> torch.Tensor:
     if width == rows:
         return weight
     return torch.cat([weight, weight.new_zeros((width - rows,) + tuple(weight.shape[1:]))]).contiguous()
+
+
+def _pad_cols(weight: torch.Tensor, width: int = 0, multiple: int = 8) -> torch.Tensor:
+    """Columns of zeros up to ``width``, or to a multiple."""
+    cols = weight.shape[1]
+    width = width or -(-cols // multiple) * multiple
+    if width <= cols:
+        return weight.contiguous()
+    return torch.cat([weight, weight.new_zeros(weight.shape[0], width - cols)], dim=1).contiguous()
 
 
 def _lowered_rows(sums: torch.Tensor, ws, dtype, num_rows: int) -> torch.Tensor:
@@ -433,6 +455,167 @@ class GatedDeltaRule(Mixer):
             scratch = ws.get(f"gated_delta.chunks{H}_{D}_{V}", (size,), torch.float32)
         kernels.gated_delta_scan(x, b, a, *rule, y, ctx.q_start, ctx.q_len, ctx.seq_slots, ctx.num_seqs, T, packed,
                                  ctx.status, chunk_scratch=scratch)
+
+
+@register_part("mixer", "selective_scan")
+class SelectiveScan(Mixer):
+    """``params``: hidden_size, inner, state_size, rank, conv_taps.  ``in.weight`` holds the rows x | z, ``low.weight`` the
+    rows low | B | C.  A request's state row holds S as [channel][state], then the convolution's last inputs."""
+
+    takes_padded_steps = True
+
+    def __init__(self, params, weights, dtype, device, position=None) -> None:
+        super().__init__(params, weights, dtype, device)
+        self.hidden_size = E = int(params["hidden_size"])
+        self.inner = I = int(params["inner"])
+        self.state_size = N = int(params["state_size"])
+        self.rank = R = int(params["rank"])
+        self.taps = int(params["conv_taps"])
+        if N > 512:
+            raise ValueError(f"state_size={N} is more than the scan kernel holds of a channel (512)")
+        if self.taps < 1:
+            raise ValueError("conv_taps must be at least 1")
+        # x | z, each padded with rows of zeros to whole 16-byte packs.
+        self.inner_padded = P = -(-I // 8) * 8
+        w_in = self.expect("in.weight", (2 * I, E))
+        self.w_in = torch.cat([_pad_rows(w_in[:I]), _pad_rows(w_in[I:])]).contiguous()
+        self.w_low = _pad_cols(_pad_rows(self.expect("low.weight", (R + 2 * N, I))))
+        self.low_width = self.w_low.shape[0]
+        self.w_dt = self.expect("dt.weight", (I, R)).contiguous()
+        # As a product of its own it reads whole rows of low, B and C against columns of zeros.
+        self.w_dt_wide = _pad_rows(_pad_cols(self.w_dt, self.low_width))
+        self.weights.pop("in.weight", None)
+        self.conv_t = self.expect("conv.weight", (I, self.taps)).to(torch.float32).t().contiguous()
+        self.conv_b = self.expect("conv.bias", (I,)).to(torch.float32).contiguous()
+        self.dt_bias = self.expect("dt.bias", (I,)).to(torch.float32).contiguous()
+        # A log2(e), formed once: the kernels' exponentials are powers of two.
+        a = -torch.exp(self.expect("a_log", (I, N)).to(torch.float64))
+        self.a2 = (a * math.log2(math.e)).to(torch.float32).contiguous()
+        self.d_skip = self.expect("d", (I,)).to(torch.float32).contiguous()
+        self.w_out = _pad_cols(self.expect("out.weight", (E, I)))
+        self.state_elems = -(-I * N // 4) * 4
+        self.conv_elems = (self.taps - 1) * I
+        kernels.mixers()
+
+    def cache_needs(self) -> CacheNeeds:
+        return CacheNeeds(state=StateSpec(shape=(-(-(self.state_elems + self.conv_elems) // 4) * 4,), dtype=torch.float32))
+
+    def forward(self, x, ctx, cache):
+        T, I, P, R, N = ctx.num_tokens, self.inner, self.inner_padded, self.rank, self.state_size
+        ws = ctx.workspace
+        if hasattr(x, "materialize"):
+            x = x.materialize()
+        proj = ws.get(f"selective.in{2 * P}", (ws.max_tokens, 2 * P), self.dtype)
+        linear(x, self.w_in, None, proj, T, status=ctx.status)
+        # (Columns behind I stay zero in both buffers: nothing writes them.)
+        u = ws.get(f"selective.x{I}_{P}", (ws.max_tokens, P), self.dtype)
+        state = cache.state
+        conv_state = state[:, self.state_elems :] if self.taps > 1 else state
+        kernels.conv_act(proj[:, :I], self.conv_t, self.conv_b, conv_state, u[:, :I], ctx.q_start, ctx.q_len, ctx.seq_slots,
+                         ctx.num_seqs, T, kernels.ACT_SILU)
+        low = ws.get(f"selective.low{self.low_width}", (ws.max_tokens, self.low_width), self.dtype)
+        linear(u, self.w_low, None, low, T, status=ctx.status)
+        y = ws.get(f"selective.y{I}_{P}", (ws.max_tokens, P), self.dtype)
+        z = proj[:, P : P + I]
+        done = ctx.single_tokens and kernels.selective_step(
+            u[:, :I], low, self.w_dt, self.dt_bias, self.a2, self.d_skip, z, y[:, :I], state[:, : self.state_elems],
+            ctx.q_start, ctx.seq_slots, ctx.num_seqs)
+        if not done:
+            dt = ws.get(f"selective.dt{P}", (ws.max_tokens, P), torch.float32)
+            linear(low, self.w_dt_wide, None, dt, T, status=ctx.status)
+            chunk = kernels.selective_chunk(T, ctx.num_seqs, I, N)
+            chunk_states = chunk_dt = None
+            if chunk:
+                # Places for the chunks (of at least 64 tokens) of any step.
+                places = ws.max_tokens // 64 + state.shape[0] + 1
+                chunk_states = ws.get(f"selective.chunk_states{I}_{N}", (places * I * N,), torch.float32)
+                chunk_dt = ws.get(f"selective.chunk_dt{I}", (places * I,), torch.float32)
+            kernels.selective_scan(u[:, :I], dt[:, :I], self.dt_bias, self.a2, low[:, R : R + 2 * N], self.d_skip, z, y[:, :I],
+                                   state[:, : self.state_elems], ctx.q_start, ctx.q_len, ctx.seq_slots, ctx.num_seqs, T,
+                                   chunk=chunk, chunk_states=chunk_states, chunk_dt=chunk_dt)
+        return product_of(y, self.w_out, ctx, T)
+
+
+@register_part("mixer", "gated_linear_attention")
+class GatedLinearAttention(Mixer):
+    """``params``: hidden_size, heads, dim, value_dim, rank, tau, eps.  ``in.weight`` holds the rows q | k | v | g | low; the
+    second half of the decay's low-rank pair is ``decay_up.weight`` with ``decay_bias``.  A request's state row holds S
+    as [head][value][key]."""
+
+    takes_padded_steps = True
+
+    def __init__(self, params, weights, dtype, device, position=None) -> None:
+        super().__init__(params, weights, dtype, device)
+        self.hidden_size = E = int(params["hidden_size"])
+        self.heads = H = int(params["heads"])
+        self.dim = D = int(params["dim"])
+        self.value_dim = V = int(params["value_dim"])
+        self.rank = R = int(params["rank"])
+        self.tau = float(params["tau"])
+        self.eps = float(params["eps"])
+        if D > 512:
+            raise ValueError(f"dim={D} is more than the kernels hold in a column's lanes (512)")
+        if not self.tau > 0.0:
+            raise ValueError(f"tau={self.tau} must be positive")
+        self.q_scale = D ** -0.5
+        keys, inner = H * D, H * V
+        self.inner, self.inner_padded = inner, -(-inner // 8) * 8
+        # q | k | v, padding to whole packs, g | low.
+        w = self.expect("in.weight", (2 * keys + 2 * inner + R, E))
+        self.g_at = -(-(2 * keys + inner) // 8) * 8
+        self.low_at = -(-(self.g_at + inner) // 8) * 8
+        self.rank_padded = -(-R // 8) * 8
+        wide = w.new_zeros(self.low_at + self.rank_padded, E)
+        wide[: 2 * keys + inner] = w[: 2 * keys + inner]
+        wide[self.g_at : self.g_at + inner] = w[2 * keys + inner : 2 * keys + 2 * inner]
+        wide[self.low_at : self.low_at + R] = w[2 * keys + 2 * inner :]
+        self.w_in = wide
+        self.in_width = wide.shape[0]
+        self.weights.pop("in.weight", None)
+        self.w_up = self.expect("decay_up.weight", (keys, R)).contiguous()
+        self.w_up_wide = _pad_rows(_pad_cols(self.w_up))
+        self.decay_bias = self.expect("decay_bias", (keys,)).to(torch.float32).contiguous()
+        self.norm_w = self.expect("norm.weight", (V,)).to(torch.float32).contiguous()
+        self.norm_all = self.norm_w.repeat(H).contiguous()
+        self.w_out = _pad_cols(self.expect("out.weight", (E, inner)))
+        self.state_elems = -(-H * V * D // 4) * 4
+        kernels.mixers()
+
+    def cache_needs(self) -> CacheNeeds:
+        return CacheNeeds(state=StateSpec(shape=(self.state_elems,), dtype=torch.float32))
+
+    def forward(self, x, ctx, cache):
+        T, H, D, V, R = ctx.num_tokens, self.heads, self.dim, self.value_dim, self.rank
+        keys, inner = H * D, self.inner
+        ws = ctx.workspace
+        if hasattr(x, "materialize"):
+            x = x.materialize()
+        proj = ws.get(f"gated_linear.in{self.in_width}", (ws.max_tokens, self.in_width), self.dtype)
+        linear(x, self.w_in, None, proj, T, status=ctx.status)
+        q, k, v = proj[:, :keys], proj[:, keys : 2 * keys], proj[:, 2 * keys : 2 * keys + inner]
+        g = proj[:, self.g_at : self.g_at + inner]
+        # (Columns behind inner stay zero: nothing writes them.)
+        normed = ws.get(f"gated_linear.normed{inner}", (ws.max_tokens, self.inner_padded), self.dtype)
+        state = cache.state
+        done = ctx.single_tokens and kernels.gated_linear_step(
+            q, k, v, proj[:, self.low_at : self.low_at + R], self.w_up, self.decay_bias, self.q_scale, self.tau, H, D, V, g,
+            self.norm_w, self.eps, normed[:, :inner], state, ctx.q_start, ctx.seq_slots, ctx.num_seqs)
+        if not done:
+            low = proj[:, self.low_at : self.low_at + self.rank_padded]
+            if self.dtype == torch.float32 or T <= SMALL_STEP_TOKENS:
+                # (The library's product takes rows with a pitch.)
+                rows = ws.get(f"gated_linear.low{self.rank_padded}", (ws.max_tokens, self.rank_padded), self.dtype)
+                kernels.act_rows(low, rows, T, kernels.ACT_NONE)
+                low = rows
+            z = ws.get(f"gated_linear.z{self.w_up_wide.shape[0]}", (ws.max_tokens, self.w_up_wide.shape[0]), torch.float32)
+            linear(low, self.w_up_wide, None, z, T, status=ctx.status)
+            size = kernels.gated_linear_scratch(ws.max_tokens, state.shape[0], H, D)
+            records = ws.get("gated_linear.records%d" % size, (size,), torch.float32)
+            y = ws.get(f"gated_linear.y{inner}", (ws.max_tokens, inner), torch.float32)
+            kernels.gated_linear_chunks(q, k, v, z[:, :keys], self.decay_bias, self.q_scale, self.tau, H, D, V, records, state,
+                                        y, ctx.q_start, ctx.q_len, ctx.seq_slots, ctx.num_seqs, T, ctx.status)
+            kernels.gated_group_norm(y, g, self.norm_all, self.eps, H, normed[:, :inner], T, gate_after=kernels.GATE_SILU)
+        return product_of(normed, self.w_out, ctx, T)
 
 
 @register_part("mixer", "side_by_side")

@@ -36,9 +36,25 @@ def stretch_slow_pairs(inv_freq: torch.Tensor, rotary_dim: int, base: float, sca
     return inv_freq / factor * ramp + inv_freq * (1.0 - ramp), 0.1 * math.log(factor) + 1.0
 
 
+def stretch_long_waves(inv_freq: torch.Tensor, scaling) -> torch.Tensor:
+    """``scaling`` = {factor, low, high, original}: with a pair's wavelength ``l = 2 pi / f`` in positions, f stays where
+    ``l < original / high``, becomes ``f / factor`` where ``l > original / low``, and between the two, with ``s =
+    (original / l - low) / (high - low)``, ``(1 - s) f / factor + s f``.  (float64.)"""
+    import math
+
+    f = inv_freq.to(torch.float64)
+    factor, low, high, original = (float(scaling[key]) for key in ("factor", "low", "high", "original"))
+    waves = 2.0 * math.pi / f
+    # (low = high: there is no range between the two.)
+    s = (original / waves - low) / (high - low) if high != low else torch.zeros_like(f)
+    mixed = (1.0 - s) * f / factor + s * f
+    return torch.where(waves < original / high, f, torch.where(waves > original / low, f / factor, mixed))
+
+
 @register_part("position", "rotary_half")
 class RotaryHalf(PositionEncoding):
-    """``scaling`` = {factor, original, fast, slow} stretches the slow pairs (``stretch_slow_pairs``;
+    """``scaling`` = {factor, original, fast, slow} stretches the slow pairs (``stretch_slow_pairs``),
+    {factor, original, low, high} those of long wavelengths (``stretch_long_waves``;
     the angles are then formed in float64).  ``layout`` tells a mixer that rotates with its own
     kernel which dims are a pair: dim i with dim i + rotary_dim / 2."""
 
@@ -63,7 +79,9 @@ class RotaryHalf(PositionEncoding):
         exponent = torch.arange(0, self.rotary_dim, 2, dtype=work) / self.rotary_dim
         inv_freq = 1.0 / (self.theta ** exponent)
         magnitude = 1.0
-        if scaling:
+        if scaling and "low" in scaling:
+            inv_freq = stretch_long_waves(inv_freq, scaling)
+        elif scaling:
             inv_freq, magnitude = stretch_slow_pairs(inv_freq, self.rotary_dim, self.theta, scaling)
         positions = torch.arange(self.max_position, dtype=work)
         if self.scaling_factor != 1.0:
