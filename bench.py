@@ -635,11 +635,11 @@ def _reference_numbers(args, ref_root):
 
 
 def run_compare(args):
-    """``--compare-designs SIZE,...``: one layer of the Peratar, Redalix, Lizizen, Mamivik and Petanex designs
-    beside one layer of the Qwen2 design at the same width, head count and feed-forward weight
+    """``--compare-designs SIZE,...``: one layer of the Peratar, Redalix, Lizizen, Mamivik, Petanex and Demavik
+    designs beside one layer of the Qwen2 design at the same width, head count and feed-forward weight
     count per token (the presets ``peratar-<size>``, ``redalix-<size>``, ``lizizen-<size>``, ``mamivik-<size>``,
-    ``petanex-<size>`` and ``<size>`` of ``velox_b200.config.presets``), random weights.  A Redalix or Petanex "layer" is the mean
-    over one period of its pattern of four layers, a Lizizen or Mamivik "layer" the mean of its two kinds.  Per
+    ``petanex-<size>``, ``demavik-<size>`` and ``<size>`` of ``velox_b200.config.presets``), random weights.  A Redalix, Petanex or
+    Demavik "layer" is the mean over one period of its pattern of four layers, a Lizizen or Mamivik "layer" the mean of its two kinds.  Per
     design and size: the time of a decode layer (``--batch`` requests behind 4,096 keys) against
     its bytes and the measured copy bandwidth, the time of a 2,048-token prompt layer against its
     operations and the measured library bf16 rate, and the time a layer spends in every kind of
@@ -655,7 +655,7 @@ def run_compare(args):
     rows = []
     for size in args.compare_designs.split(","):
         for name in (size, "peratar-" + size, "redalix-" + size, "lizizen-" + size, "mamivik-" + size,
-                     "petanex-" + size):
+                     "petanex-" + size, "demavik-" + size):
             if args.designs and name.split("-")[0] not in args.designs.split(",") and not (
                     "-" not in name and "qwen2" in args.designs.split(",")):
                 continue
@@ -675,7 +675,8 @@ def run_compare(args):
                 "design": ("Peratar" if name.startswith("peratar-") else "Redalix" if name.startswith("redalix-")
                            else "Lizizen" if name.startswith("lizizen-")
                            else "Mamivik" if name.startswith("mamivik-")
-                           else "Petanex" if name.startswith("petanex-") else "Qwen2"),
+                           else "Petanex" if name.startswith("petanex-")
+                           else "Demavik" if name.startswith("demavik-") else "Qwen2"),
                 "size": size,
                 "decode": {"batch": args.batch, "keys": keys, "us_per_layer": round(decode_s * 1e6, 1),
                            "layer_bytes": weights + cached, "us_by_bytes": round((weights + cached) / (peaks["hbm_gbs"] * 1e9) * 1e6, 1),
@@ -709,10 +710,10 @@ def main():
     parser.add_argument("--impl", default="own", choices=["own", "reference"])
     parser.add_argument("--no-points", dest="points", action="store_false", help="skip the batch 1 / 64 points")
     parser.add_argument("--compare-designs", default=None, metavar="SIZE,...",
-                        help="instead of the benchmark: one layer of the Peratar, Redalix, Lizizen, Mamivik and Petanex designs beside one of the "
+                        help="instead of the benchmark: one layer of the Peratar, Redalix, Lizizen, Mamivik, Petanex and Demavik designs beside one of the "
                              "Qwen2 design at the named sizes (0.5b, 1.5b, 3b), decode and prefill")
     parser.add_argument("--designs", default=None, metavar="NAME,...",
-                        help="with --compare-designs: only these designs (qwen2, peratar, redalix, lizizen, mamivik, petanex)")
+                        help="with --compare-designs: only these designs (qwen2, peratar, redalix, lizizen, mamivik, petanex, demavik)")
     args = parser.parse_args()
     world = int(os.environ.get("WORLD_SIZE", "1"))
     if args.gpus > 1 or world > 1:

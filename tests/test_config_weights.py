@@ -87,6 +87,9 @@ def test_named_model_sizes_are_configurations_of_the_architecture():
         if name.startswith("petanex-") or name == "tiny-x":
             assert arch.name == "Petanex" and len(typed.layers) == len(cfg["layers"])
             continue
+        if name.startswith("demavik-") or name == "tiny-d":
+            assert arch.name == "Demavik" and len(typed.layers) == len(cfg["layers"])
+            continue
         assert arch.name == "Qwen2ForCausalLM"
         c = Qwen2Config.from_dict(cfg)
         assert c.num_attention_heads % c.num_key_value_heads == 0

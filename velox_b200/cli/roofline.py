@@ -249,6 +249,49 @@ def _petanex_layer(entry: Dict, width: int, tokens: int, batch: int, context: in
     return 2 * weights, cache, flops
 
 
+def _is_demavik(config_json: Dict) -> bool:
+    return config_json.get("architecture") == "Demavik" or "Demavik" in (config_json.get("architectures") or [])
+
+
+def _demavik_layer(entry: Dict, width: int, tokens: int, batch: int, context: int):
+    """(bytes of weights read, bytes of cache and state touched, operations) of one Demavik layer for
+    ``tokens`` new tokens of each of ``batch`` sequences behind ``context`` keys.  Recurrent states are read and
+    written once a step; an entry costs five operations per token in gated linear attention and seven in the
+    selective scan (its exponential as one); of the experts as many are read as the step's tokens can name."""
+    from ..config.model_config import GatedLinearConfig
+    from ..models.demavik import default_rank
+
+    kind, m = entry["type"], entry["mixer"]
+    rows = batch * tokens
+    cache, flops = 0, 0.0
+    if kind == "mamba1":
+        inner, states, rank = m["inner"], m["state"], m["dt_rank"]
+        weights = 2 * inner * width + (rank + 2 * states) * inner + inner * rank + width * inner
+        cache += batch * inner * (2 * states + m["conv"]) * 4
+        flops += 7.0 * rows * inner * states
+    elif kind == "gla":
+        keys, inner = m["heads"] * m["dim"], m["heads"] * m["vdim"]
+        rank = default_rank(GatedLinearConfig(m["heads"], m["dim"], m["vdim"], m["tau"]))
+        weights = (2 * keys + 2 * inner + rank) * width + keys * rank + width * inner
+        cache += batch * inner * m["dim"] * 2 * 4
+        flops += 5.0 * rows * inner * m["dim"]
+    else:
+        heads, kv = m["heads"], m["kv_heads"]
+        weights = heads * m["dim"] * width + width * heads * m["vdim"]
+        if m.get("kv_from") is None:
+            weights += kv * (m["dim"] + m["vdim"]) * width
+        pairs = tokens * (context + (tokens + 1) / 2.0)
+        cache += batch * (context + tokens) * kv * (m["dim"] + m["vdim"]) * 2
+        flops += 2.0 * batch * pairs * heads * (m["dim"] + m["vdim"])
+    flops += 2.0 * rows * weights
+    mlp = entry.get("mlp")
+    if mlp is not None:
+        experts, top, ff = mlp["router"]["experts"], mlp["router"]["top"], mlp["expert"]["ff"]
+        weights += min(experts, rows * top) * 3 * ff * width + experts * width
+        flops += 2.0 * rows * (top * 3 * ff + experts) * width
+    return 2 * weights, cache, flops
+
+
 def _listed_layer(config_json: Dict):
     """The per-layer accounting of a design whose layers differ in kind, or None."""
     if _is_redalix(config_json):
@@ -259,6 +302,8 @@ def _listed_layer(config_json: Dict):
         return _mamivik_layer
     if _is_petanex(config_json):
         return _petanex_layer
+    if _is_demavik(config_json):
+        return _demavik_layer
     return None
 
 

@@ -258,7 +258,56 @@ def _petanex_tiny() -> Dict[str, Any]:
             "token_side": {"dim": 24}, "layers": layers, "max_position_embeddings": 512}
 
 
+def _demavik(like: str, experts: int = 32, top: int = 4, buckets: int = 16384) -> Dict[str, Any]:
+    """A Demavik configuration with the width, attention head counts, layer count, vocabulary and feed-forward weights
+    per token of the named Qwen2.5 size.  Its layers repeat the pattern mamba1 (twice the width in channels, 16
+    states, a sixteenth of the width as step-size rank), gla (four heads of an eighth of the width by a
+    quarter), attention, attention with the keys of the layer before; every layer has ``experts`` experts,
+    ``top`` per token."""
+    base = MODEL_SIZES[like]
+    width, heads, kv_heads = base["hidden_size"], base["num_attention_heads"], base["num_key_value_heads"]
+    head = base.get("head_dim") or width // heads
+    part = max(64, base["intermediate_size"] // top // 64 * 64)
+    moe = {"kind": "moe", "expert": {"ff": part}, "router": {"experts": experts, "top": top}}
+    attention = {"heads": heads, "kv_heads": kv_heads, "dim": head, "vdim": head, "scale": head ** -0.5,
+                 "rot": {"base": 500000.0, "dims": head,
+                         "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}
+    pattern = [
+        {"type": "mamba1", "mixer": {"inner": 2 * width, "state": 16, "dt_rank": width // 16, "conv": 4}, "mlp": moe},
+        {"type": "gla", "mixer": {"heads": 4, "dim": width // 8, "vdim": width // 4, "tau": 16.0}, "mlp": moe},
+        {"type": "attention", "mixer": attention, "mlp": moe},
+        {"type": "attention", "mixer": attention, "mlp": moe},
+    ]
+    entries = [copy.deepcopy(pattern[index % len(pattern)]) for index in range(base["num_hidden_layers"])]
+    for index, entry in enumerate(entries):
+        if index % len(pattern) == 3:
+            entry["mixer"]["kv_from"] = index - 1
+    return {"architecture": "Demavik", "vocab": base["vocab_size"], "width": width, "norm": {"eps": 1e-6},
+            "residual_mult": 0.25, "embedding": {"scale": 1.0, "bigram": {"buckets": buckets, "mul_prev": 31, "mul_cur": 17}},
+            "layers": entries, "max_position_embeddings": base["max_position_embeddings"]}
+
+
+def _demavik_tiny() -> Dict[str, Any]:
+    """A tiny Demavik configuration for smoke runs of the command lines: one layer of each kind, one that reads another's
+    keys, one without feed-forward."""
+    attention = {"heads": 4, "kv_heads": 2, "dim": 16, "vdim": 32, "scale": 0.25, "rot": {"base": 5000.0, "dims": 8}}
+    moe = {"kind": "moe", "expert": {"ff": 48}, "router": {"experts": 6, "top": 2}}
+    layers = [
+        {"type": "gla", "mixer": {"heads": 2, "dim": 32, "vdim": 16, "tau": 8.0}, "mlp": moe},
+        {"type": "attention", "mixer": attention, "mlp": None},
+        {"type": "mamba1", "mixer": {"inner": 160, "state": 8, "dt_rank": 8, "conv": 3}, "mlp": moe},
+        {"type": "attention", "mixer": dict(attention, kv_from=1), "mlp": moe},
+    ]
+    return {"architecture": "Demavik", "vocab": 384, "width": 128, "norm": {"eps": 1e-5}, "residual_mult": 0.4,
+            "embedding": {"scale": 2.0, "bigram": {"buckets": 211, "mul_prev": 5, "mul_cur": 3}}, "layers": layers,
+            "max_position_embeddings": 512}
+
+
 MODEL_SIZES.update({
+    "tiny-d": _demavik_tiny(),
+    "demavik-0.5b": _demavik("0.5b"),
+    "demavik-1.5b": _demavik("1.5b"),
+    "demavik-3b": _demavik("3b"),
     "tiny-x": _petanex_tiny(),
     "petanex-0.5b": _petanex("0.5b"),
     "petanex-1.5b": _petanex("1.5b"),
