@@ -76,11 +76,11 @@ SMALL = config(64, 120, [
 ODD = config(100, 331, [
     layer("attention", attn(3, 1, 14, 30, 0.4, rot(10, 30.0)), moe(5, 2, 17)),
     layer("mamba1", mamba(54, 5, 3, 2), None),
-    layer("gla", gla(3, 10, 7, 1.0), moe(7, 1, 20)),
+    layer("gla", gla(3, 10, 7, 1.0), moe(7, 2, 20)),
     layer("attention", attn(6, 1, 14, 30, 0.3, rot(10, 30.0), kv_from=0), moe(2, 2, 9)),
     layer("gla", gla(1, 6, 15, 3.5), None),
     layer("mamba1", mamba(130, 1, 1, 1), moe(9, 4, 12)),
-], eps=1e-5, mult=0.6, scale=1.3, bigram=None)
+], eps=1e-5, mult=0.3, scale=1.3, bigram=None)
 
 # Sizes near a real model's.
 WIDE = config(256, 500, [

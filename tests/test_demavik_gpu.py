@@ -780,36 +780,35 @@ def test_a_key_that_takes_nearly_all_weight(tmp_path, dtype, shared, ask_at, nee
 def test_a_write_is_recalled_hundreds_of_tokens_later(tmp_path, kind, dtype):
     """A state that hardly decays and into which hardly any token but one writes: what that one wrote 600 tokens ago
     is read by a query made to ask for it, across chunks, portions, pages and decoded tokens."""
+    mixer = dc.gla(2, 16, 24, 16.0) if kind == "gla" else dc.mamba(48, 6, 4, 2)
+    cfg, tensors = model_of([dc.layer(kind, mixer, None)])
+    # one coordinate of the stream is the marker's alone, one the asker's
+    tensors["embed"][:, :2] = 0.0
+    tensors["embed"][MARKER, 0] = tensors["embed"][ASKER, 1] = 2.0
+    gen = torch.Generator().manual_seed(5)
+    p = "l0.mix."
     if kind == "gla":
-        cfg, tensors = model_of([dc.layer("gla", dc.gla(2, 16, 24, 16.0), None)])
-        tensors["l0.mix.a2"].zero_()
-        tensors["l0.mix.a2.b"].fill_(14.0)
-        em, ea = stream_row(tensors, MARKER), stream_row(tensors, ASKER)
-        tensors["l0.mix.k"] = 0.02 * tensors["l0.mix.k"]
-        tensors["l0.mix.q"] = 0.05 * tensors["l0.mix.q"]
-        key = torch.randn(32, generator=torch.Generator().manual_seed(1))
-        tensors["l0.mix.k"] += 6.0 * torch.outer(key, em) / float(em @ em)
-        tensors["l0.mix.q"] += 6.0 * torch.outer(key, ea) / float(ea @ ea)
+        tensors[p + "a2"].zero_()
+        tensors[p + "a2.b"].fill_(14.0)
+        key = torch.randn(32, generator=gen)
+        tensors[p + "k"], tensors[p + "q"] = 0.01 * tensors[p + "k"], 0.05 * tensors[p + "q"]
+        tensors[p + "k"][:, 0], tensors[p + "q"][:, 1] = key, key
     else:
-        cfg, tensors = model_of([dc.layer("mamba1", dc.mamba(48, 6, 4, 2), None)])
-        # the marker's step size is large, the others' next to nothing; B is the marker's, C the asker's
-        em, ea = stream_row(tensors, MARKER), stream_row(tensors, ASKER)
-        p = "l0.mix."
+        # the first two channels read those coordinates; the marker's step size is large, the others' next to nothing
         tensors[p + "conv"][:, 0] = 0.0
         tensors[p + "conv"][:, 1] = 1.0
         tensors[p + "conv.b"].zero_()
         tensors[p + "A_log"].fill_(-6.0)
         tensors[p + "D"].zero_()
-        x = torch.nn.functional.silu(tensors[p + "in"][:48] @ em)
+        tensors[p + "in"][:2] = 0.0
+        tensors[p + "in"][0, 0] = tensors[p + "in"][1, 1] = 2.0
         tensors[p + "x"].zero_()
-        tensors[p + "x"][0] = 12.0 * x / float(x @ x)
+        tensors[p + "x"][0, 0] = 1.5
+        tensors[p + "x"][4:10, 0] = 0.2 * torch.randn(6, generator=gen)
+        tensors[p + "x"][10:16, 1] = 0.2 * torch.randn(6, generator=gen)
         tensors[p + "dt"].zero_()
         tensors[p + "dt"][:, 0] = 1.0
         tensors[p + "dt.b"].fill_(-9.0)
-        gen = torch.Generator().manual_seed(5)
-        tensors[p + "x"][4:10] = torch.outer(torch.randn(6, generator=gen), x) / float(x @ x)
-        xa = torch.nn.functional.silu(tensors[p + "in"][:48] @ ea)
-        tensors[p + "x"][10:16] = torch.outer(torch.randn(6, generator=gen), xa) / float(xa @ xa)
     folder, tensors = written(tmp_path, cfg, tensors)
     length, needle_at, ask_at = 700, 40, 655
     tokens, without = pointed_prompt(length, needle_at, ask_at, seed=3)
@@ -837,6 +836,8 @@ def test_the_edges_of_the_convolution(tmp_path, conv, dtype):
     cfg, tensors = model_of([dc.layer("mamba1", dc.mamba(48, 4, 4, conv), None)])
     tensors["l0.mix.dt.b"].fill_(60.0)
     tensors["l0.mix.A_log"].fill_(2.0)
+    tensors["l0.mix.x"][8:12] = tensors["l0.mix.x"][4:8]   # C = B: the state's share cannot nearly cancel the input's
+    tensors["l0.mix.D"].fill_(1.0)
     tensors["l0.mix.conv"][:, 0] = 1.5 * torch.sign(tensors["l0.mix.conv"][:, 0])
     folder, tensors = written(tmp_path, cfg, tensors)
     tokens = random_prompts(VOCAB, [40], seed=8)[0]
@@ -861,6 +862,8 @@ def test_the_edge_of_the_pair_embedding(tmp_path, dtype):
     cfg, tensors = model_of([dc.layer("mamba1", dc.mamba(48, 4, 4, 1), None)], bigram=(61, 12, 5))
     tensors["l0.mix.dt.b"].fill_(60.0)
     tensors["l0.mix.A_log"].fill_(2.0)
+    tensors["l0.mix.x"][8:12] = tensors["l0.mix.x"][4:8]   # C = B: the state's share cannot nearly cancel the input's
+    tensors["l0.mix.D"].fill_(1.0)
     folder, tensors = written(tmp_path, cfg, tensors)
     tokens = random_prompts(VOCAB, [40], seed=18)[0]
     at = 25

@@ -292,14 +292,35 @@ gated_linear_chunk_kernel(GatedLinear p, const float* __restrict__ z, long long 
   }
 }
 
-// Warps 0-3 carry the state (a thread: four rows of four columns for every 128 rows, in registers; a copy in shared
-// memory for the products that read it), warps 4-7 make o from the state as it was.  Records come in by
+// W rows of the state at a time, as a thread holds them and as they lie in shared memory.
+template <int W>
+__device__ __forceinline__ void load_rows(const float* p, float (&v)[W]) {
+  if constexpr (W == 4) {
+    const float4 f = *reinterpret_cast<const float4*>(p);
+    v[0] = f.x, v[1] = f.y, v[2] = f.z, v[3] = f.w;
+  } else if constexpr (W == 2) {
+    const float2 f = *reinterpret_cast<const float2*>(p);
+    v[0] = f.x, v[1] = f.y;
+  } else {
+    v[0] = *p;
+  }
+}
+template <int W>
+__device__ __forceinline__ void store_rows(float* p, const float (&v)[W]) {
+  if constexpr (W == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+  else if constexpr (W == 2) *reinterpret_cast<float2*>(p) = make_float2(v[0], v[1]);
+  else *p = v[0];
+}
+
+// Warps 0-3 carry the state (a thread: NV rows of four columns, in registers; a copy in shared memory for the
+// products that read it), warps 4-7 make o from the state as it was.  Records come in by
 // bulk copies, STAGES of them under way; the values' tile comes through registers.
 template <typename T, int NV, int STAGES>
 __global__ void __launch_bounds__(LP_THREADS)
 gated_linear_pass_kernel(GatedLinear p, const float* __restrict__ records, float* __restrict__ state,
                          long long state_stride, float* __restrict__ out, long long out_stride, int* status) {
-  constexpr int KD = 32 * NV, SP = KD + 4, NJ = (KD + 127) / 128, VP = LP_COLS + 4;
+  constexpr int KD = 32 * NV, SP = KD + 4, VP = LP_COLS + 4;
+  constexpr int W = NV % 4 == 0 ? 4 : NV % 2 == 0 ? 2 : 1, NJ = NV / W;  // rows lane * W + 32 W j of a lane
   constexpr int REC = 2 * LC * KD + LC * LC_BP + KD;
   extern __shared__ __align__(16) float gl_s[];
   float* S_s = gl_s + STAGES * REC;       // [LP_COLS][SP]
@@ -352,18 +373,17 @@ gated_linear_pass_kernel(GatedLinear p, const float* __restrict__ records, float
   put_values(0);
   float* st = state + (size_t)slot * state_stride + (size_t)h * Dv * Dk;
   const int my_cols = (warp & 3) * 4;
-  float S[NJ][4][4];
+  float S[NJ][4][W];
   if (warp < 4) {
 #pragma unroll
     for (int j = 0; j < NJ; ++j) {
-      const int k0 = lane * 4 + 128 * j;
+      const int k0 = lane * W + 32 * W * j;
 #pragma unroll
       for (int c = 0; c < 4; ++c) {
         const int col = tile * LP_COLS + my_cols + c;
 #pragma unroll
-        for (int e = 0; e < 4; ++e) S[j][c][e] = col < Dv && k0 + e < Dk ? st[(size_t)col * Dk + k0 + e] : 0.f;
-        if (k0 < KD)
-          *reinterpret_cast<float4*>(S_s + (my_cols + c) * SP + k0) = make_float4(S[j][c][0], S[j][c][1], S[j][c][2], S[j][c][3]);
+        for (int e = 0; e < W; ++e) S[j][c][e] = col < Dv && k0 + e < Dk ? st[(size_t)col * Dk + k0 + e] : 0.f;
+        store_rows<W>(S_s + (my_cols + c) * SP + k0, S[j][c]);
       }
     }
   }
@@ -380,28 +400,25 @@ gated_linear_pass_kernel(GatedLinear p, const float* __restrict__ records, float
       const float* pv = buf + 2 * LC * KD + LC * LC_BP;
 #pragma unroll
       for (int j = 0; j < NJ; ++j) {
-        const int k0 = lane * 4 + 128 * j;
-        if (k0 >= KD) break;
-        const float4 decay = *reinterpret_cast<const float4*>(pv + k0);
+        float decay[W];
+        load_rows<W>(pv + lane * W + 32 * W * j, decay);
 #pragma unroll
-        for (int c = 0; c < 4; ++c) S[j][c][0] *= decay.x, S[j][c][1] *= decay.y, S[j][c][2] *= decay.z, S[j][c][3] *= decay.w;
+        for (int c = 0; c < 4; ++c)
+#pragma unroll
+          for (int e = 0; e < W; ++e) S[j][c][e] *= decay[e];
       }
 #pragma unroll 4
       for (int i = 0; i < LC; ++i) {
-        const float4 vv = *reinterpret_cast<const float4*>(v_s + i * VP + my_cols);
-        const float v[4] = {vv.x, vv.y, vv.z, vv.w};
+        float v[4];
+        load_rows<4>(v_s + i * VP + my_cols, v);
 #pragma unroll
         for (int j = 0; j < NJ; ++j) {
-          const int k0 = lane * 4 + 128 * j;
-          if (k0 >= KD) break;
-          const float4 kv = *reinterpret_cast<const float4*>(kh + i * KD + k0);
+          float kv[W];
+          load_rows<W>(kh + i * KD + lane * W + 32 * W * j, kv);
 #pragma unroll
-          for (int c = 0; c < 4; ++c) {
-            S[j][c][0] = fmaf(kv.x, v[c], S[j][c][0]);
-            S[j][c][1] = fmaf(kv.y, v[c], S[j][c][1]);
-            S[j][c][2] = fmaf(kv.z, v[c], S[j][c][2]);
-            S[j][c][3] = fmaf(kv.w, v[c], S[j][c][3]);
-          }
+          for (int c = 0; c < 4; ++c)
+#pragma unroll
+            for (int e = 0; e < W; ++e) S[j][c][e] = fmaf(kv[e], v[c], S[j][c][e]);
         }
       }
     } else {
@@ -426,6 +443,22 @@ gated_linear_pass_kernel(GatedLinear p, const float* __restrict__ records, float
           }
         }
       }
+      {
+        // The chunk's own share, B times the values: four of its 32 tokens a lane, in the same sums.
+        const float* b = buf + 2 * LC * KD + (size_t)(warp - 4) * 8 * LC_BP + 4 * kg;
+        float vv[4][4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) load_rows<4>(v_s + (4 * kg + e) * VP + c0, vv[e]);
+#pragma unroll
+        for (int r = 0; r < 8; ++r) {
+          float bv[4];
+          load_rows<4>(b + r * LC_BP, bv);
+#pragma unroll
+          for (int e = 0; e < 4; ++e)
+#pragma unroll
+            for (int c = 0; c < 4; ++c) acc[4 * r + c] = fmaf(bv[e], vv[e][c], acc[4 * r + c]);
+        }
+      }
       // Over the eight lanes, lane kg ending with row kg of the eight.
 #pragma unroll
       for (int off = 4; off > 0; off >>= 1) {
@@ -438,20 +471,6 @@ gated_linear_pass_kernel(GatedLinear p, const float* __restrict__ records, float
         }
       }
       const int row = (warp - 4) * 8 + kg;
-      const float* b = buf + 2 * LC * KD + row * LC_BP;
-#pragma unroll
-      for (int j = 0; j < LC; j += 4) {
-        const float4 bv = *reinterpret_cast<const float4*>(b + j);
-        const float bj[4] = {bv.x, bv.y, bv.z, bv.w};
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const float4 vv = *reinterpret_cast<const float4*>(v_s + (j + e) * VP + c0);
-          acc[0] = fmaf(bj[e], vv.x, acc[0]);
-          acc[1] = fmaf(bj[e], vv.y, acc[1]);
-          acc[2] = fmaf(bj[e], vv.z, acc[2]);
-          acc[3] = fmaf(bj[e], vv.w, acc[3]);
-        }
-      }
       const int token = chunk * LC + row;
       if (token < n) {
         float* dst = out + (size_t)(start + token) * out_stride + (size_t)h * Dv + tile * LP_COLS + c0;
@@ -465,13 +484,9 @@ gated_linear_pass_kernel(GatedLinear p, const float* __restrict__ records, float
     if (chunk + 1 < chunks) put_values(chunk + 1);
     if (warp < 4) {
 #pragma unroll
-      for (int j = 0; j < NJ; ++j) {
-        const int k0 = lane * 4 + 128 * j;
-        if (k0 >= KD) break;
+      for (int j = 0; j < NJ; ++j)
 #pragma unroll
-        for (int c = 0; c < 4; ++c)
-          *reinterpret_cast<float4*>(S_s + (my_cols + c) * SP + k0) = make_float4(S[j][c][0], S[j][c][1], S[j][c][2], S[j][c][3]);
-      }
+        for (int c = 0; c < 4; ++c) store_rows<W>(S_s + (my_cols + c) * SP + lane * W + 32 * W * j, S[j][c]);
     }
     __syncthreads();
   }
@@ -479,12 +494,12 @@ gated_linear_pass_kernel(GatedLinear p, const float* __restrict__ records, float
   if (warp < 4) {
 #pragma unroll
     for (int j = 0; j < NJ; ++j) {
-      const int k0 = lane * 4 + 128 * j;
+      const int k0 = lane * W + 32 * W * j;
 #pragma unroll
       for (int c = 0; c < 4; ++c) {
         const int col = tile * LP_COLS + my_cols + c;
 #pragma unroll
-        for (int e = 0; e < 4; ++e)
+        for (int e = 0; e < W; ++e)
           if (col < Dv && k0 + e < Dk) st[(size_t)col * Dk + k0 + e] = S[j][c][e];
       }
     }

@@ -157,17 +157,50 @@ conv_act_kernel(const T* __restrict__ x, long long x_stride, int channels, int t
 }
 
 // ---------------------------------------------------------------------------------------------
-// The scan.  Channels never meet, so a block takes SS_THREADS / L channels of one sequence: L lanes of a warp share
-// a channel, each with NS of its states in registers.  Tokens come SS_TC at a time through shared memory (the next
-// ones are on their way while these are used); a token of no step size and no input (behind the end) changes
-// nothing.  Four tokens' shares of y meet by shuffles at once, each ending in another lane.
+// The scan.  Channels never meet, so a block takes CB channels of one sequence.  Its scan warps do nothing else: L lanes of
+// a warp share a channel, each with NS of its states in registers, and four tokens' shares of y meet by shuffles at
+// once, each ending in another lane.  Two pairs of helper warps bring tile after tile of tokens into shared memory (step
+// sizes through their softplus), each pair every other one so that its loads have two tiles' time to arrive, and
+// turn the sums of a tile that is done into outputs.  A token of no step size and no input (behind the end) changes nothing.
 //
 // Mode 0: a whole sequence in one block, from the slot's state.  Long portions of models with few channels run in
 // chunks of `chunk` tokens side by side: every chunk from a zero state, keeping its last state and the sum of
 // its step sizes (mode 1; a chunk's whole decay is exp(A sum dt)); the chunks' starting states in order
 // (selective_combine_kernel); every chunk again from its starting state, writing y (mode 2).  The chunks of
 // sequence s lie at places q_start[s] / chunk + s + c.
-constexpr int SS_THREADS = 128;
+constexpr int SS_THREADS = 128;  // of the one-token kernel
+constexpr int SS_HELPERS = 64;   // of a tile
+__host__ __device__ constexpr int ss_scan_threads(int L) { return L <= 4 ? 64 : 128; }
+__host__ __device__ constexpr int ss_tile(int L, int NP) { return NP >= 256 ? 4 : NP >= 128 || L == 1 ? 8 : 16; }
+
+// PV neighbouring values of a row.
+template <typename T, int PV>
+struct PairOf;
+template <typename T>
+struct PairOf<T, 1> {
+  T v;
+  __device__ __forceinline__ void load(const T* p) { v = *p; }
+  __device__ __forceinline__ float get(int) const { return to_float(v); }
+  static __device__ __forceinline__ void store(T* p, const float (&f)[1]) { *p = from_float<T>(f[0]); }
+};
+template <>
+struct PairOf<float, 2> {
+  float2 v;
+  __device__ __forceinline__ void load(const float* p) { v = *reinterpret_cast<const float2*>(p); }
+  __device__ __forceinline__ float get(int e) const { return e == 0 ? v.x : v.y; }
+  static __device__ __forceinline__ void store(float* p, const float (&f)[2]) {
+    *reinterpret_cast<float2*>(p) = make_float2(f[0], f[1]);
+  }
+};
+template <>
+struct PairOf<__nv_bfloat16, 2> {
+  uint32_t v;
+  __device__ __forceinline__ void load(const __nv_bfloat16* p) { v = *reinterpret_cast<const uint32_t*>(p); }
+  __device__ __forceinline__ float get(int e) const { return __uint_as_float(e == 0 ? v << 16 : v & 0xffff0000u); }
+  static __device__ __forceinline__ void store(__nv_bfloat16* p, const float (&f)[2]) {
+    *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(f[0], f[1]);
+  }
+};
 
 struct SelectiveScan {
   const void* x;           // [tokens, inner] in the compute dtype
@@ -191,23 +224,39 @@ struct SelectiveScan {
   float* chunk_dt;         // [places][inner]
 };
 
-template <typename T, int L, int NS, int MODE>
-__global__ void __launch_bounds__(SS_THREADS) selective_scan_kernel(SelectiveScan p) {
-  constexpr int CB = SS_THREADS / L, NP = L * NS;
-  constexpr int TC = NP >= 256 ? 4 : NP >= 128 ? 8 : 16;
-  constexpr int BUF = 2 * TC * CB + 2 * TC * NP;
-  constexpr int CH_PER = (TC * CB + SS_THREADS - 1) / SS_THREADS;
-  constexpr int BC_PER = 2 * TC * NP / SS_THREADS > 0 ? (2 * TC * NP + SS_THREADS - 1) / SS_THREADS : 1;
-  extern __shared__ __align__(16) float ss_s[];
+template <typename T, int L, int NS, int MODE, bool VEC>
+__global__ void __launch_bounds__(ss_scan_threads(L) + 2 * SS_HELPERS) selective_scan_kernel(SelectiveScan p) {
+  constexpr int SCAN = ss_scan_threads(L), CB = SCAN / L, NP = L * NS, TC = ss_tile(L, NP);
+  constexpr int BUF = 2 * TC * CB + 2 * TC * NP;  // dt, dt x, then B | C of every token
+  // A helper's places of a tile: CH_PER tokens of PV neighbouring channels, STEP tokens apart.  VEC: channels in
+  // pairs, and the B | C rows in packs of sixteen bytes, where sizes and alignment allow it.
+  constexpr int PV = VEC ? 2 : 1, LANES = CB / PV, STEP = SS_HELPERS / LANES;
+  constexpr int CH_PER = (TC + STEP - 1) / STEP;
+  constexpr int BC_PER = 2 * TC * NP / SS_HELPERS;       // values a helper
+  static_assert(SS_HELPERS % CB == 0 && 2 * TC * NP % SS_HELPERS == 0, "a helper keeps to its channels");
+  extern __shared__ __align__(16) float ss_s[];  // two buffers, then y of two tiles [TC][CB]
+  float* y_s = ss_s + 2 * BUF;
   allow_dependents();
-  const int tid = threadIdx.x, r = tid % L, ch = tid / L;
-  const int c0 = blockIdx.x * CB, c = c0 + ch, s = blockIdx.y;
-  const bool live = c < p.inner;
+  const int tid = threadIdx.x, c0 = blockIdx.x * CB, s = blockIdx.y;
+  const bool scans = tid < SCAN;
+  const int r = tid % L, ch = tid / L, c = c0 + ch;  // of a scanning thread
+  const bool live = scans && c < p.inner;
   float a2[NS], S[NS];
+  if (scans) {
 #pragma unroll
-  for (int k = 0; k < NS; ++k) {
-    const int n = r * NS + k;
-    a2[k] = live && n < p.N ? p.a2[(size_t)c * p.N + n] : 0.f;
+    for (int k = 0; k < NS; ++k) {
+      const int n = r * NS + k;
+      a2[k] = live && n < p.N ? p.a2[(size_t)c * p.N + n] : 0.f;
+    }
+  }
+  const int pair = (tid - SCAN) / SS_HELPERS, helper = (tid - SCAN) % SS_HELPERS;  // of a helper
+  const int q = scans ? 0 : (helper % LANES) * PV, k0 = scans ? 0 : helper / LANES;
+  const bool q_ok = !scans && c0 + q < p.inner;
+  float bias[PV], skip[PV];
+#pragma unroll
+  for (int e = 0; e < PV; ++e) {
+    bias[e] = q_ok ? p.dt_bias[c0 + q + e] : 0.f;
+    skip[e] = q_ok ? p.d_skip[c0 + q + e] : 0.f;
   }
   grid_dependency_wait();
   const int seq_tokens = p.q_len[s], seq_start = p.q_start[s];
@@ -218,148 +267,221 @@ __global__ void __launch_bounds__(SS_THREADS) selective_scan_kernel(SelectiveSca
   const size_t place = MODE == 0 ? 0 : (size_t)(seq_start / p.chunk + s) + blockIdx.z;
   float* st = MODE == 0 ? p.state + (size_t)p.seq_slots[s] * p.state_stride : p.chunk_states + place * p.inner * p.N;
   st += (size_t)c * p.N;
-#pragma unroll
-  for (int k = 0; k < NS; ++k) {
-    const int n = r * NS + k;
-    S[k] = MODE != 1 && live && n < p.N ? st[n] : 0.f;
-  }
-  float dt_sum = 0.f;
-  const T* x = (const T*)p.x + start * p.x_stride + c0;
-  const T* z = (const T*)p.z + start * p.z_stride + c0;
-  const T* bc = (const T*)p.bc + start * p.bc_stride;
-  const float* dtl = p.dt + start * p.dt_stride + c0;
-  T* out = (T*)p.out + start * p.out_stride + c0;
-  // A thread's places of a tile: (token, channel) pairs tid + u SS_THREADS, the channel the same for all of them
-  // where a tile's width divides the block.
-  T pre_x[CH_PER], pre_z[CH_PER], pre_bc[BC_PER], cur_x[CH_PER], cur_z[CH_PER];
-  float pre_dt[CH_PER];
-  auto fetch = [&](int i0) {
-    const int tc = min(TC, n_tok - i0);
-#pragma unroll
-    for (int u = 0; u < CH_PER; ++u) {
-      const int idx = tid + u * SS_THREADS, k = idx / CB, q = idx - k * CB;
-      const bool ok = k < tc && c0 + q < p.inner;
-      // Loads from valid places, used or not: behind conditions they would be waited for one by one.
-      const size_t row = (size_t)(i0 + (ok ? k : 0));
-      const int col = ok ? q : 0;
-      pre_x[u] = x[row * p.x_stride + col];
-      pre_dt[u] = dtl[row * p.dt_stride + col];
-      if (MODE != 1) pre_z[u] = z[row * p.z_stride + col];
-    }
-#pragma unroll
-    for (int u = 0; u < BC_PER; ++u) {
-      const int idx = tid + u * SS_THREADS, k = idx / (2 * NP), j = idx - k * (2 * NP), arr = j / NP, n = j - arr * NP;
-      const bool ok = k < tc && n < p.N;
-      pre_bc[u] = bc[(size_t)(i0 + (ok ? k : 0)) * p.bc_stride + (ok ? arr * p.N + n : 0)];
-    }
-  };
-  auto put = [&](float* buf, int i0) {
-    const int tc = min(TC, n_tok - i0);
-#pragma unroll
-    for (int u = 0; u < CH_PER; ++u) {
-      const int idx = tid + u * SS_THREADS, k = idx / CB, q = idx - k * CB;
-      const bool ok = k < tc && c0 + q < p.inner;
-      if (idx < TC * CB) {
-        const float dt = ok ? softplus_for<T>(pre_dt[u] + p.dt_bias[c0 + (ok ? q : 0)]) : 0.f;
-        buf[idx] = dt;
-        buf[TC * CB + idx] = ok ? dt * to_float(pre_x[u]) : 0.f;
-      }
-      cur_x[u] = pre_x[u];
-      if (MODE != 1) cur_z[u] = pre_z[u];
-    }
-#pragma unroll
-    for (int u = 0; u < BC_PER; ++u) {
-      const int idx = tid + u * SS_THREADS, k = idx / (2 * NP), j = idx - k * (2 * NP), arr = j / NP, n = j - arr * NP;
-      if (idx < 2 * TC * NP) buf[2 * TC * CB + idx] = k < tc && n < p.N ? to_float(pre_bc[u]) : 0.f;
-    }
-  };
-  fetch(0);
-  put(ss_s, 0);
-  __syncthreads();
-  int which = 0;
-  for (int i0 = 0; i0 < n_tok; i0 += TC) {
-    float* buf = ss_s + which * BUF;
-    const bool more = i0 + TC < n_tok;
-    if (more) fetch(i0 + TC);
-    float* dt_s = buf + ch;               // [TC][CB]; a token's place takes its y when the step size is used
-    const float* dx_s = buf + TC * CB + ch;
-    const float* bc_s = buf + 2 * TC * CB + r * NS;  // [TC][B NP | C NP]
-#pragma unroll 1
-    for (int k0 = 0; k0 < TC; k0 += 4) {
-      float y[4];
-#pragma unroll
-      for (int kk = 0; kk < 4; ++kk) {
-        const int k = k0 + kk;
-        const float dt = dt_s[k * CB], dx = dx_s[k * CB];
-        if (MODE == 1) dt_sum += dt;
-        float b[NS], cc[NS];
-#pragma unroll
-        for (int j = 0; j < NS; j += 4) {
-          const float4 bv = *reinterpret_cast<const float4*>(bc_s + k * 2 * NP + j);
-          b[j] = bv.x, b[j + 1] = bv.y, b[j + 2] = bv.z, b[j + 3] = bv.w;
-          if (MODE != 1) {
-            const float4 cv = *reinterpret_cast<const float4*>(bc_s + k * 2 * NP + NP + j);
-            cc[j] = cv.x, cc[j + 1] = cv.y, cc[j + 2] = cv.z, cc[j + 3] = cv.w;
-          }
-        }
-        float acc = 0.f;
-#pragma unroll
-        for (int j = 0; j < NS; ++j) {
-          S[j] = fmaf(pow2_for<T>(dt * a2[j]), S[j], dx * b[j]);
-          if (MODE != 1) acc = fmaf(S[j], cc[j], acc);
-        }
-        y[kk] = acc;
-      }
-      if (MODE != 1) {
-        // Two tokens stay with each lane of a pair, then one with each lane of four.
-        int token = 0;
-        if (L >= 2) {
-          const bool up = (r & 1) != 0;
-#pragma unroll
-          for (int i = 0; i < 2; ++i) {
-            const float give = up ? y[i] : y[i + 2], keep = up ? y[i + 2] : y[i];
-            y[i] = keep + __shfl_xor_sync(0xffffffffu, give, 1);
-          }
-          token = up ? 2 : 0;
-        }
-        if (L >= 4) {
-          const bool up = (r & 2) != 0;
-          const float give = up ? y[0] : y[1], keep = up ? y[1] : y[0];
-          y[0] = keep + __shfl_xor_sync(0xffffffffu, give, 2);
-          token += up ? 1 : 0;
-#pragma unroll
-          for (int off = 4; off < L; off <<= 1) y[0] += __shfl_xor_sync(0xffffffffu, y[0], off);
-        }
-        constexpr int OWN = L >= 4 ? 1 : 4 / L;
-        if (L <= 4 || r < 4) {
-#pragma unroll
-          for (int i = 0; i < OWN; ++i) dt_s[(k0 + token + i) * CB] = y[i];
-        }
-      }
-    }
-    if (MODE != 1) {
-      __syncthreads();
-#pragma unroll
-      for (int u = 0; u < CH_PER; ++u) {
-        const int idx = tid + u * SS_THREADS, k = idx / CB, q = idx - k * CB;
-        if (idx < TC * CB && i0 + k < n_tok && c0 + q < p.inner)
-          out[(size_t)(i0 + k) * p.out_stride + q] =
-              from_float<T>(fmaf(p.d_skip[c0 + q], to_float(cur_x[u]), buf[idx]) * silu_for<T>(to_float(cur_z[u])));
-      }
-    }
-    if (more) put(ss_s + (which ^ 1) * BUF, i0 + TC);
-    __syncthreads();  // the next tokens are in place, and these may be overwritten
-    which ^= 1;
-  }
-  if (MODE == 2) return;
-  if (live) {
+  const int tiles = (n_tok + TC - 1) / TC;
+  if (scans) {
 #pragma unroll
     for (int k = 0; k < NS; ++k) {
       const int n = r * NS + k;
-      if (n < p.N) st[n] = S[k];
+      S[k] = MODE != 1 && live && n < p.N ? st[n] : 0.f;
     }
-    if (MODE == 1 && r == 0) p.chunk_dt[place * p.inner + c] = dt_sum;
+    float dt_sum = 0.f;
+    __syncthreads();  // the first tile is there
+    for (int i = 0; i < tiles; ++i) {
+      const float* buf = ss_s + (i & 1) * BUF;
+      const float* dt_s = buf + ch;
+      const float* dx_s = buf + TC * CB + ch;
+      const float* bc_s = buf + 2 * TC * CB + r * NS;
+      float* y_out = y_s + (i & 1) * TC * CB + ch;
+      // A tile's sums stay in registers until its last token: a store among the loads of later tokens would hold
+      // them up (it could be to the same place).
+      constexpr int OWN = L >= 4 ? 1 : 4 / L;
+      float sums[TC / 4][OWN];
+      int token = 0;
+#pragma unroll
+      for (int g = 0; g < TC; g += 4) {
+        float y[4];
+#pragma unroll
+        for (int kk = 0; kk < 4; ++kk) {
+          const int k = g + kk;
+          const float dt = dt_s[k * CB], dx = dx_s[k * CB];
+          if (MODE == 1) dt_sum += dt;
+          float b[NS], cc[NS];
+#pragma unroll
+          for (int j = 0; j < NS; j += 4) {
+            const float4 bv = *reinterpret_cast<const float4*>(bc_s + k * 2 * NP + j);
+            b[j] = bv.x, b[j + 1] = bv.y, b[j + 2] = bv.z, b[j + 3] = bv.w;
+            if (MODE != 1) {
+              const float4 cv = *reinterpret_cast<const float4*>(bc_s + k * 2 * NP + NP + j);
+              cc[j] = cv.x, cc[j + 1] = cv.y, cc[j + 2] = cv.z, cc[j + 3] = cv.w;
+            }
+          }
+          float acc = 0.f;
+#pragma unroll
+          for (int j = 0; j < NS; ++j) {
+            S[j] = fmaf(pow2_for<T>(dt * a2[j]), S[j], dx * b[j]);
+            if (MODE != 1) acc = fmaf(S[j], cc[j], acc);
+          }
+          y[kk] = acc;
+        }
+        if (MODE != 1) {
+          // Two tokens stay with each lane of a pair, then one with each lane of four.
+          if (L >= 2) {
+            const bool up = (r & 1) != 0;
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+              const float give = up ? y[e] : y[e + 2], keep = up ? y[e + 2] : y[e];
+              y[e] = keep + __shfl_xor_sync(0xffffffffu, give, 1);
+            }
+            token = up ? 2 : 0;
+          }
+          if (L >= 4) {
+            const bool up = (r & 2) != 0;
+            const float give = up ? y[0] : y[1], keep = up ? y[1] : y[0];
+            y[0] = keep + __shfl_xor_sync(0xffffffffu, give, 2);
+            token += up ? 1 : 0;
+            if constexpr (L > 4) {
+#pragma unroll
+              for (int off = 4; off < L; off <<= 1) y[0] += __shfl_xor_sync(0xffffffffu, y[0], off);
+            }
+          }
+#pragma unroll
+          for (int e = 0; e < OWN; ++e) sums[g / 4][e] = y[e];
+        }
+      }
+      if (MODE != 1 && (L <= 4 || r < 4)) {
+#pragma unroll
+        for (int g = 0; g < TC; g += 4)
+#pragma unroll
+          for (int e = 0; e < OWN; ++e) y_out[(g + token + e) * CB] = sums[g / 4][e];
+      }
+      __syncthreads();
+    }
+    if (MODE != 2 && live) {
+#pragma unroll
+      for (int k = 0; k < NS; ++k) {
+        const int n = r * NS + k;
+        if (n < p.N) st[n] = S[k];
+      }
+      if (MODE == 1 && r == 0) p.chunk_dt[place * p.inner + c] = dt_sum;
+    }
+    return;
   }
+  // Helpers.  Loads go to valid places, used or not: behind conditions they would be waited for one by one.
+  const int col = q_ok ? q : 0;
+  const T* x = (const T*)p.x + start * p.x_stride + c0 + col;
+  const T* z = (const T*)p.z + start * p.z_stride + c0 + col;
+  const T* bc = (const T*)p.bc + start * p.bc_stride;
+  const float* dtl = p.dt + start * p.dt_stride + c0 + col;
+  T* out = (T*)p.out + start * p.out_stride + c0 + col;
+  typedef PairOf<T, PV> Pair;
+  Pair in_x[CH_PER], in_z[CH_PER], past_x[CH_PER], past_z[CH_PER];  // on their way; of the tile that is scanned
+  PairOf<float, PV> in_dt[CH_PER];
+  T in_bc[VEC ? 1 : BC_PER];
+  // Sixteen-byte packs of a tile's B | C rows: a helper's are at the same places of every tile.
+  constexpr int PACK = 16 / (int)sizeof(T), PACK_PER = VEC ? (2 * TC * NP / PACK + SS_HELPERS - 1) / SS_HELPERS : 1;
+  RowVec<T, VEC ? PACK : 1> in_packs[PACK_PER];
+  int pack_token[PACK_PER], pack_col[PACK_PER], pack_at[PACK_PER];
+  if constexpr (VEC) {
+    const int per_row = 2 * p.N / PACK, packs = TC * per_row;
+#pragma unroll
+    for (int u = 0; u < PACK_PER; ++u) {
+      const int at = helper + u * SS_HELPERS, k = min(at, packs - 1) / per_row, j = (min(at, packs - 1) - k * per_row) * PACK;
+      pack_token[u] = k;
+      pack_col[u] = j;
+      pack_at[u] = at < packs ? k * 2 * NP + (j < p.N ? j : NP + j - p.N) : -1;
+    }
+    // What lies behind N states of a row is never written again.
+    if (p.N < NP)
+      for (int idx = tid - SCAN; idx < 4 * TC * NP; idx += 2 * SS_HELPERS)
+        if ((idx & (NP - 1)) >= p.N) ss_s[(idx / (2 * TC * NP)) * BUF + 2 * TC * CB + idx % (2 * TC * NP)] = 0.f;
+  }
+  auto fetch = [&](int i) {
+    const int i0 = i * TC;
+#pragma unroll
+    for (int u = 0; u < CH_PER; ++u) {
+      const size_t row = (size_t)min(i0 + k0 + u * STEP, n_tok - 1);
+      in_x[u].load(x + row * p.x_stride);
+      in_dt[u].load(dtl + row * p.dt_stride);
+      if (MODE != 1) in_z[u].load(z + row * p.z_stride);
+    }
+    if constexpr (VEC) {
+#pragma unroll
+      for (int u = 0; u < PACK_PER; ++u) {
+        in_packs[u].load(bc + (size_t)min(i0 + pack_token[u], n_tok - 1) * p.bc_stride + pack_col[u]);
+      }
+    } else {
+#pragma unroll
+      for (int u = 0; u < BC_PER; ++u) {
+        const int idx = helper + u * SS_HELPERS, k = idx / (2 * NP), j = idx - k * (2 * NP), arr = j / NP, n = j - arr * NP;
+        if (MODE == 1 && NP >= SS_HELPERS && arr == 1) continue;
+        in_bc[u] = bc[(size_t)min(i0 + k, n_tok - 1) * p.bc_stride + arr * p.N + min(n, p.N - 1)];
+      }
+    }
+  };
+  auto put = [&](int i) {
+    const int i0 = i * TC;
+    float* buf = ss_s + (i & 1) * BUF;
+#pragma unroll
+    for (int u = 0; u < CH_PER; ++u) {
+      const int k = k0 + u * STEP;
+      const bool ok = q_ok && i0 + k < n_tok;
+      if (k < TC) {
+        float dt[PV], dx[PV];
+#pragma unroll
+        for (int e = 0; e < PV; ++e) {
+          dt[e] = ok ? softplus_for<T>(in_dt[u].get(e) + bias[e]) : 0.f;
+          dx[e] = ok ? dt[e] * in_x[u].get(e) : 0.f;
+        }
+        PairOf<float, PV>::store(buf + k * CB + q, dt);
+        PairOf<float, PV>::store(buf + TC * CB + k * CB + q, dx);
+      }
+    }
+    float* bc_out = buf + 2 * TC * CB;
+    if constexpr (VEC) {
+#pragma unroll
+      for (int u = 0; u < PACK_PER; ++u) {
+        if (pack_at[u] >= 0) {
+          float v[PACK];
+          in_packs[u].get(v);
+#pragma unroll
+          for (int e = 0; e < PACK; e += 4)
+            *reinterpret_cast<float4*>(bc_out + pack_at[u] + e) = make_float4(v[e], v[e + 1], v[e + 2], v[e + 3]);
+        }
+      }
+    } else {
+#pragma unroll
+      for (int u = 0; u < BC_PER; ++u) {
+        const int idx = helper + u * SS_HELPERS, k = idx / (2 * NP), j = idx - k * (2 * NP), n = j & (NP - 1);
+        if (MODE == 1 && NP >= SS_HELPERS && j >= NP) continue;
+        bc_out[idx] = i0 + k < n_tok && n < p.N ? to_float(in_bc[u]) : 0.f;
+      }
+    }
+  };
+  auto finish = [&](int i) {
+#pragma unroll
+    for (int u = 0; u < CH_PER; ++u) {
+      const int k = k0 + u * STEP;
+      if (k < TC && q_ok && i * TC + k < n_tok) {
+        float y[PV];
+#pragma unroll
+        for (int e = 0; e < PV; ++e)
+          y[e] = fmaf(skip[e], past_x[u].get(e), y_s[(i & 1) * TC * CB + k * CB + q + e]) * silu_for<T>(past_z[u].get(e));
+        Pair::store(out + (size_t)(i * TC + k) * p.out_stride, y);
+      }
+    }
+  };
+  // A pair's turn: the sums of its tile before, then its next tile into the other buffer, then the loads of the one
+  // after that.  (A tile of a token behind the end has dt = dx = 0: what B and C hold there does not matter.)
+  auto turn = [&](int i) {  // tile i is scanned; i + 1 is put in place, i - 1 is done
+    if (MODE != 1 && i > 0) finish(i - 1);
+    if (i + 1 < tiles) {
+      put(i + 1);
+#pragma unroll
+      for (int u = 0; u < CH_PER; ++u) {
+        past_x[u] = in_x[u];
+        if (MODE != 1) past_z[u] = in_z[u];
+      }
+      if (i + 3 < tiles) fetch(i + 3);
+    }
+  };
+  if (pair < tiles) fetch(pair);
+  if (pair == 0) turn(-1);
+  __syncthreads();
+  for (int i = 0; i < tiles; ++i) {
+    if (((i + 1) & 1) == pair) turn(i);
+    __syncthreads();
+  }
+  if (MODE != 1 && ((tiles - 1) & 1) == pair) finish(tiles - 1);
 }
 
 // Per sequence: the states its chunks start from, in order (each in the place of the chunk's own last state), and
@@ -376,12 +498,25 @@ __global__ void selective_combine_kernel(SelectiveScan p) {
     const size_t c = e / p.N;
     const float a2 = p.a2[e];
     float* st = p.state + (size_t)p.seq_slots[s] * p.state_stride + e;
+    float* at = p.chunk_states + first * total + e;
+    const float* dt = p.chunk_dt + first * p.inner + c;
     float S = *st;
-    for (int k = 0; k < chunks; ++k) {
-      float* at = p.chunk_states + (first + k) * total + e;
-      const float own = *at;
-      *at = S;
-      S = fmaf(pow2_for<T>(a2 * p.chunk_dt[(first + k) * p.inner + c]), S, own);
+    for (int k = 0; k < chunks; k += 8) {
+      // Eight chunks' values are under way together.
+      float own[8], decay[8];
+#pragma unroll
+      for (int u = 0; u < 8; ++u) {
+        const size_t at_k = (size_t)min(k + u, chunks - 1);
+        own[u] = at[at_k * total];
+        decay[u] = dt[at_k * p.inner];
+      }
+#pragma unroll
+      for (int u = 0; u < 8; ++u) {
+        if (k + u < chunks) {
+          at[(size_t)(k + u) * total] = S;
+          S = fmaf(pow2_for<T>(a2 * decay[u]), S, own[u]);
+        }
+      }
     }
     *st = S;
   }
@@ -524,32 +659,46 @@ VX_API int vx_conv_act(const void* x, int dtype, long long x_stride, int channel
   return (int)cudaGetLastError();
 }
 
-template <typename T, int L, int NS>
+template <typename T, int L, int NS, bool VEC>
 static int launch_selective_scan(const SelectiveScan& p, int num_seqs, int num_tokens, cudaStream_t stream) {
-  constexpr int CB = SS_THREADS / L, NP = L * NS, TC = NP >= 256 ? 4 : NP >= 128 ? 8 : 16;
-  constexpr size_t smem = sizeof(float) * 2 * (2 * TC * CB + 2 * TC * NP);
+  constexpr int THREADS = ss_scan_threads(L) + 2 * SS_HELPERS, CB = ss_scan_threads(L) / L, NP = L * NS, TC = ss_tile(L, NP);
+  constexpr size_t smem = sizeof(float) * 2 * (3 * TC * CB + 2 * TC * NP);
   static bool configured = false;
   if (smem > 48 * 1024 && !configured) {
-    cudaError_t e = cudaFuncSetAttribute(selective_scan_kernel<T, L, NS, 0>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaError_t e = cudaFuncSetAttribute(selective_scan_kernel<T, L, NS, 0, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e == cudaSuccess)
-      e = cudaFuncSetAttribute(selective_scan_kernel<T, L, NS, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+      e = cudaFuncSetAttribute(selective_scan_kernel<T, L, NS, 1, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e == cudaSuccess)
-      e = cudaFuncSetAttribute(selective_scan_kernel<T, L, NS, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+      e = cudaFuncSetAttribute(selective_scan_kernel<T, L, NS, 2, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
     configured = true;
   }
   const int blocks = (p.inner + CB - 1) / CB;
   if (p.chunk <= 0 || num_tokens <= p.chunk) {
-    launch_pdl(selective_scan_kernel<T, L, NS, 0>, dim3(blocks, num_seqs), dim3(SS_THREADS), smem, stream, p);
+    launch_pdl(selective_scan_kernel<T, L, NS, 0, VEC>, dim3(blocks, num_seqs), dim3(THREADS), smem, stream, p);
     return (int)cudaGetLastError();
   }
   const dim3 grid(blocks, num_seqs, (num_tokens + p.chunk - 1) / p.chunk);
-  launch_pdl(selective_scan_kernel<T, L, NS, 1>, grid, dim3(SS_THREADS), smem, stream, p);
+  launch_pdl(selective_scan_kernel<T, L, NS, 1, VEC>, grid, dim3(THREADS), smem, stream, p);
   int cblocks = (int)(((size_t)p.inner * p.N + 255) / 256);
   if (cblocks > 148 * 8) cblocks = 148 * 8;
   launch_pdl(selective_combine_kernel<T>, dim3(cblocks, num_seqs), dim3(256), 0, stream, p);
-  launch_pdl(selective_scan_kernel<T, L, NS, 2>, grid, dim3(SS_THREADS), smem, stream, p);
+  launch_pdl(selective_scan_kernel<T, L, NS, 2, VEC>, grid, dim3(THREADS), smem, stream, p);
   return (int)cudaGetLastError();
+}
+
+template <typename T, int L, int NS>
+static int choose_selective_scan(const SelectiveScan& p, int num_seqs, int num_tokens, cudaStream_t stream) {
+  if constexpr (NS == 4 && L <= 16) {
+    // Channels in pairs, B and C in sixteen-byte packs: sizes, pitches and pointers allow it.
+    const int pack = 16 / (int)sizeof(T);
+    const bool vec = p.N % pack == 0 && p.inner % 2 == 0 && p.x_stride % 2 == 0 && p.z_stride % 2 == 0 && p.out_stride % 2 == 0 &&
+                     p.dt_stride % 2 == 0 && p.bc_stride % pack == 0 && (reinterpret_cast<uintptr_t>(p.bc) & 15) == 0 &&
+                     ((reinterpret_cast<uintptr_t>(p.x) | reinterpret_cast<uintptr_t>(p.z) | reinterpret_cast<uintptr_t>(p.out) |
+                       reinterpret_cast<uintptr_t>(p.dt)) & 7) == 0;
+    if (vec) return launch_selective_scan<T, L, NS, true>(p, num_seqs, num_tokens, stream);
+  }
+  return launch_selective_scan<T, L, NS, false>(p, num_seqs, num_tokens, stream);
 }
 
 // The most states of a channel the kernels hold.
@@ -557,12 +706,8 @@ VX_API int vx_selective_max_state() { return 512; }
 
 // Channels of one block of the scan, for the caller's choice of chunks.
 VX_API int vx_selective_block_channels(int N) {
-  if (N <= 4) return SS_THREADS;
-  if (N <= 8) return SS_THREADS / 2;
-  if (N <= 16) return SS_THREADS / 4;
-  if (N <= 32) return SS_THREADS / 8;
-  if (N <= 64) return SS_THREADS / 16;
-  return SS_THREADS / 32;
+  const int L = N <= 4 ? 1 : N <= 8 ? 2 : N <= 16 ? 4 : N <= 32 ? 8 : N <= 64 ? 16 : 32;
+  return ss_scan_threads(L) / L;
 }
 
 #define VX_SELECTIVE_SIZES(CALL)   \
@@ -588,7 +733,7 @@ VX_API int vx_selective_scan(const void* x, int dtype, long long x_stride, const
   if (chunk_states == nullptr || chunk_dt == nullptr) chunk = 0;
   const SelectiveScan p = {x, x_stride, dt, dt_stride, dt_bias, a2, bc, bc_stride, d_skip, z, z_stride, out, out_stride,
                            state, state_stride, inner, N, chunk, q_start, q_len, seq_slots, chunk_states, chunk_dt};
-#define VX_SCAN_CALL(L, NS) VX_BY_DTYPE(dtype, return (launch_selective_scan<T, L, NS>(p, num_seqs, num_tokens, stream)))
+#define VX_SCAN_CALL(L, NS) VX_BY_DTYPE(dtype, return (choose_selective_scan<T, L, NS>(p, num_seqs, num_tokens, stream)))
   VX_SELECTIVE_SIZES(VX_SCAN_CALL)
 #undef VX_SCAN_CALL
 }

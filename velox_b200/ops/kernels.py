@@ -1842,10 +1842,10 @@ def selective_chunk(num_tokens: int, num_seqs: int, inner: int, states: int) -> 
     """Tokens of a chunk with which ``selective_scan`` should cut a step's portions (0: not at all): chunks run
     side by side but make every decay twice, so they pay only where whole sequences leave SMs without work."""
     blocks = -(-inner // int(mixers().vx_selective_block_channels(states))) * num_seqs
-    if num_tokens < 256 or 2 * blocks > 148:
+    if num_tokens < 256 or blocks > 128:
         return 0
-    # About two blocks an SM, in chunks of at least 64 tokens.
-    return max(64, -(-num_tokens * blocks // (2 * 148 * 16)) * 16)
+    # About six blocks an SM, in chunks of at least 64 tokens.
+    return max(64, -(-num_tokens * blocks // (6 * 148 * 16)) * 16)
 
 
 def selective_scan(x, dt, dt_bias, a2, bc, d_skip, z, out, state, q_start, q_len, seq_slots, num_seqs, num_tokens,
