@@ -163,6 +163,7 @@ class ScanCase:
         state[spare] = 7.0
         a2 = (-torch.exp(self.a_log.double()) * np.log2(np.e)).float().contiguous().cuda()
         bias, d, w_dt = self.bias.cuda(), self.d.cuda(), self.w_dt.contiguous().cuda()
+        status = torch.zeros(4, dtype=torch.int32).cuda()
         got = [np.zeros((n, I)) for n in self.lengths]
         for spans, T, q_start, q_len, seq_slots in Steps(self.lengths, cuts, slots):
             x, z, low = take(self.x, spans), take(self.z, spans), take(self.low, spans)
@@ -178,8 +179,9 @@ class ScanCase:
                     scratch = dict(chunk=chunk, chunk_states=torch.full((places * I * N,), np.nan).cuda(),
                                    chunk_dt=torch.full((places * I,), np.nan).cuda())
                 k.selective_scan(xz[:, :I], dt, bias, a2, low[:, R:], d, xz[:, I:], out, state, q_start, q_len, seq_slots,
-                                 len(spans), T, **scratch)
+                                 len(spans), T, status, **scratch)
             give(got, spans, out)
+        assert int(status[0]) == 0
         assert bool((state[spare] == 7.0).all()), "another slot's state has changed"
         return got, [num(state[slot, : I * N].view(I, N)) for slot in slots]
 

@@ -358,16 +358,17 @@ gated_linear_pass_kernel(GatedLinear p, const float* __restrict__ records, float
   const T* values = (const T*)p.v + (size_t)start * p.stride + (size_t)h * Dv + tile * LP_COLS;
   const int v_col = tid % LP_COLS, v_row = tid / LP_COLS;  // and v_row + 16
   const bool v_ok = tile * LP_COLS + v_col < Dv;
-  float v0, v1;
+  T v0, v1;  // as stored: they are looked at only when the chunk before is done
   auto fetch_values = [&](int c) {
-    const int i0 = c * LC + v_row, i1 = i0 + LC / 2;
-    v0 = v_ok && i0 < n ? to_float(values[(size_t)i0 * p.stride + v_col]) : 0.f;
-    v1 = v_ok && i1 < n ? to_float(values[(size_t)i1 * p.stride + v_col]) : 0.f;
+    const int i0 = c * LC + v_row, col = v_ok ? v_col : 0;
+    v0 = values[(size_t)min(i0, n - 1) * p.stride + col];
+    v1 = values[(size_t)min(i0 + LC / 2, n - 1) * p.stride + col];
   };
   auto put_values = [&](int c) {
+    const int i0 = c * LC + v_row;
     float* dst = V_s + (c & 1) * LC * VP + v_row * VP + v_col;
-    dst[0] = v0;
-    dst[LC / 2 * VP] = v1;
+    dst[0] = v_ok && i0 < n ? to_float(v0) : 0.f;
+    dst[LC / 2 * VP] = v_ok && i0 + LC / 2 < n ? to_float(v1) : 0.f;
   };
   fetch_values(0);
   put_values(0);

@@ -16,7 +16,7 @@
 
 namespace vx {
 
-// Sixteen bytes of a row as floats, or one value.
+// Sixteen bytes of a row as floats.
 template <typename T, int V>
 struct RowVec;
 template <>
@@ -24,9 +24,6 @@ struct RowVec<float, 4> {
   float4 raw;
   __device__ __forceinline__ void load(const float* p) { raw = *reinterpret_cast<const float4*>(p); }
   __device__ __forceinline__ void get(float (&v)[4]) const { v[0] = raw.x, v[1] = raw.y, v[2] = raw.z, v[3] = raw.w; }
-  static __device__ __forceinline__ void store(float* p, const float (&v)[4]) {
-    *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
-  }
 };
 template <>
 struct RowVec<__nv_bfloat16, 8> {
@@ -40,28 +37,43 @@ struct RowVec<__nv_bfloat16, 8> {
       v[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
     }
   }
-  static __device__ __forceinline__ void store(__nv_bfloat16* p, const float (&v)[8]) {
-    uint32_t w[4];
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      const __nv_bfloat162 h = __floats2bfloat162_rn(v[2 * i], v[2 * i + 1]);
-      w[i] = *reinterpret_cast<const uint32_t*>(&h);
-    }
-    *reinterpret_cast<uint4*>(p) = make_uint4(w[0], w[1], w[2], w[3]);
-  }
 };
 template <typename T>
-struct RowVec<T, 1> {
-  T raw;
-  __device__ __forceinline__ void load(const T* p) { raw = *p; }
-  __device__ __forceinline__ void get(float (&v)[1]) const { v[0] = to_float(raw); }
-  static __device__ __forceinline__ void store(T* p, const float (&v)[1]) { *p = from_float<T>(v[0]); }
+struct RowVec<T, 1> {};
+
+// PV neighbouring values of a row.
+template <typename T, int PV>
+struct PairOf;
+template <typename T>
+struct PairOf<T, 1> {
+  T v;
+  __device__ __forceinline__ void load(const T* p) { v = *p; }
+  __device__ __forceinline__ float get(int) const { return to_float(v); }
+  static __device__ __forceinline__ void store(T* p, const float (&f)[1]) { *p = from_float<T>(f[0]); }
+};
+template <>
+struct PairOf<float, 2> {
+  float2 v;
+  __device__ __forceinline__ void load(const float* p) { v = *reinterpret_cast<const float2*>(p); }
+  __device__ __forceinline__ float get(int e) const { return e == 0 ? v.x : v.y; }
+  static __device__ __forceinline__ void store(float* p, const float (&f)[2]) {
+    *reinterpret_cast<float2*>(p) = make_float2(f[0], f[1]);
+  }
+};
+template <>
+struct PairOf<__nv_bfloat16, 2> {
+  uint32_t v;
+  __device__ __forceinline__ void load(const __nv_bfloat16* p) { v = *reinterpret_cast<const uint32_t*>(p); }
+  __device__ __forceinline__ float get(int e) const { return __uint_as_float(e == 0 ? v << 16 : v & 0xffff0000u); }
+  static __device__ __forceinline__ void store(__nv_bfloat16* p, const float (&f)[2]) {
+    *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(f[0], f[1]);
+  }
 };
 
 // ---------------------------------------------------------------------------------------------
 // out_t = act(bias + sum_k w[k] x_(t - taps + 1 + k)) per channel.  state[slot][m][c], m = 0 .. taps - 2, is the
 // input taps - 1 - m positions before the portion's first token (zero before the sequence's start).  w_t
-// [taps][channels].  A thread takes V channels of a tile of CA_TILE tokens; only the first tile of a
+// [taps][channels].  A thread takes V neighbouring channels of a tile of CA_TILE tokens; only the first tile of a
 // portion reads the state (CA_TILE >= taps - 1, or one tile holds the portion), and the same thread then
 // writes the state that the portion leaves.
 constexpr int CA_TILE = 8;
@@ -94,16 +106,17 @@ conv_act_kernel(const T* __restrict__ x, long long x_stride, int channels, int t
 #pragma unroll
       for (int v = 0; v < V; ++v) w[k][v] = at >= 0 ? w_t[(size_t)at * channels + c0 + v] : 0.f;
     }
-    RowVec<T, V> raw[CA_TILE];
+    PairOf<T, V> raw[CA_TILE];
 #pragma unroll
     for (int i = 0; i < CA_TILE; ++i) raw[i].load(xc + (size_t)min(lo + i, hi - 1) * x_stride);
 #pragma unroll
     for (int m = 0; m < TAPS - 1; ++m) {
       const int j = lo - (TAPS - 1) + m;  // place of this input in the portion
       if (j >= 0) {
-        RowVec<T, V> r;
+        PairOf<T, V> r;
         r.load(xc + (size_t)j * x_stride);
-        r.get(win[m]);
+#pragma unroll
+        for (int v = 0; v < V; ++v) win[m][v] = r.get(v);
       } else {
         const int at = taps - 1 + j;
 #pragma unroll
@@ -113,19 +126,19 @@ conv_act_kernel(const T* __restrict__ x, long long x_stride, int channels, int t
 #pragma unroll
     for (int i = 0; i < CA_TILE; ++i) {
       if (lo + i < hi) {
-        float now[V], acc[V];
-        raw[i].get(now);
+        float acc[V];
 #pragma unroll
         for (int v = 0; v < V; ++v) {
-          float a = fmaf(w[TAPS - 1][v], now[v], b[v]);
+          const float now = raw[i].get(v);
+          float a = fmaf(w[TAPS - 1][v], now, b[v]);
 #pragma unroll
           for (int k = 0; k < TAPS - 1; ++k) a = fmaf(w[k][v], win[k][v], a);
           acc[v] = act_for<T>(a, act);
 #pragma unroll
           for (int k = 0; k + 1 < TAPS - 1; ++k) win[k][v] = win[k + 1][v];
-          win[TAPS - 2][v] = now[v];
+          win[TAPS - 2][v] = now;
         }
-        RowVec<T, V>::store(oc + (size_t)(lo + i) * out_stride, acc);
+        PairOf<T, V>::store(oc + (size_t)(lo + i) * out_stride, acc);
       }
     }
   } else {
@@ -143,11 +156,12 @@ conv_act_kernel(const T* __restrict__ x, long long x_stride, int channels, int t
       }
 #pragma unroll
       for (int v = 0; v < V; ++v) acc[v] = act_for<T>(acc[v], act);
-      RowVec<T, V>::store(oc + (size_t)i * out_stride, acc);
+      PairOf<T, V>::store(oc + (size_t)i * out_stride, acc);
     }
   }
   if (lo != 0) return;
   // What the portion leaves; ascending m: what is read lies at or behind what has been written.
+#pragma unroll 1
   for (int m = 0; m < taps - 1; ++m) {
     const int j = n - (taps - 1) + m;
 #pragma unroll
@@ -159,9 +173,10 @@ conv_act_kernel(const T* __restrict__ x, long long x_stride, int channels, int t
 // ---------------------------------------------------------------------------------------------
 // The scan.  Channels never meet, so a block takes CB channels of one sequence.  Its scan warps do nothing else: L lanes of
 // a warp share a channel, each with NS of its states in registers, and four tokens' shares of y meet by shuffles at
-// once, each ending in another lane.  Two pairs of helper warps bring tile after tile of tokens into shared memory (step
-// sizes through their softplus), each pair every other one so that its loads have two tiles' time to arrive, and
-// turn the sums of a tile that is done into outputs.  A token of no step size and no input (behind the end) changes nothing.
+// once, each ending in another lane.  Four helper warps, each for every fourth tile of tokens, bring a tile into a shared
+// buffer of its own (step sizes through their softplus), ask for the one four tiles on, wait until the tile has
+// been scanned and turn its sums into outputs: a tile's way through its warp may take three times as long as
+// its scan.  Scan warps and helpers meet at two barriers per buffer.  A token of no step size and no input (behind the end) changes nothing.
 //
 // Mode 0: a whole sequence in one block, from the slot's state.  Long portions of models with few channels run in
 // chunks of `chunk` tokens side by side: every chunk from a zero state, keeping its last state and the sum of
@@ -169,38 +184,9 @@ conv_act_kernel(const T* __restrict__ x, long long x_stride, int channels, int t
 // (selective_combine_kernel); every chunk again from its starting state, writing y (mode 2).  The chunks of
 // sequence s lie at places q_start[s] / chunk + s + c.
 constexpr int SS_THREADS = 128;  // of the one-token kernel
-constexpr int SS_HELPERS = 64;   // of a tile
-__host__ __device__ constexpr int ss_scan_threads(int L) { return L <= 4 ? 64 : 128; }
+constexpr int SS_HELPERS = 32, SS_GROUPS = 4;  // helpers of a tile (a warp), and tiles that are looked after side by side
+__host__ __device__ constexpr int ss_scan_threads(int L) { return L == 1 ? 32 : L <= 4 ? 64 : 128; }
 __host__ __device__ constexpr int ss_tile(int L, int NP) { return NP >= 256 ? 4 : NP >= 128 || L == 1 ? 8 : 16; }
-
-// PV neighbouring values of a row.
-template <typename T, int PV>
-struct PairOf;
-template <typename T>
-struct PairOf<T, 1> {
-  T v;
-  __device__ __forceinline__ void load(const T* p) { v = *p; }
-  __device__ __forceinline__ float get(int) const { return to_float(v); }
-  static __device__ __forceinline__ void store(T* p, const float (&f)[1]) { *p = from_float<T>(f[0]); }
-};
-template <>
-struct PairOf<float, 2> {
-  float2 v;
-  __device__ __forceinline__ void load(const float* p) { v = *reinterpret_cast<const float2*>(p); }
-  __device__ __forceinline__ float get(int e) const { return e == 0 ? v.x : v.y; }
-  static __device__ __forceinline__ void store(float* p, const float (&f)[2]) {
-    *reinterpret_cast<float2*>(p) = make_float2(f[0], f[1]);
-  }
-};
-template <>
-struct PairOf<__nv_bfloat16, 2> {
-  uint32_t v;
-  __device__ __forceinline__ void load(const __nv_bfloat16* p) { v = *reinterpret_cast<const uint32_t*>(p); }
-  __device__ __forceinline__ float get(int e) const { return __uint_as_float(e == 0 ? v << 16 : v & 0xffff0000u); }
-  static __device__ __forceinline__ void store(__nv_bfloat16* p, const float (&f)[2]) {
-    *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(f[0], f[1]);
-  }
-};
 
 struct SelectiveScan {
   const void* x;           // [tokens, inner] in the compute dtype
@@ -222,10 +208,11 @@ struct SelectiveScan {
   const int *q_start, *q_len, *seq_slots;
   float* chunk_states;     // [places][inner, N]
   float* chunk_dt;         // [places][inner]
+  int* status;
 };
 
 template <typename T, int L, int NS, int MODE, bool VEC>
-__global__ void __launch_bounds__(ss_scan_threads(L) + 2 * SS_HELPERS) selective_scan_kernel(SelectiveScan p) {
+__global__ void __launch_bounds__(ss_scan_threads(L) + SS_GROUPS * SS_HELPERS) selective_scan_kernel(SelectiveScan p) {
   constexpr int SCAN = ss_scan_threads(L), CB = SCAN / L, NP = L * NS, TC = ss_tile(L, NP);
   constexpr int BUF = 2 * TC * CB + 2 * TC * NP;  // dt, dt x, then B | C of every token
   // A helper's places of a tile: CH_PER tokens of PV neighbouring channels, STEP tokens apart.  VEC: channels in
@@ -234,8 +221,9 @@ __global__ void __launch_bounds__(ss_scan_threads(L) + 2 * SS_HELPERS) selective
   constexpr int CH_PER = (TC + STEP - 1) / STEP;
   constexpr int BC_PER = 2 * TC * NP / SS_HELPERS;       // values a helper
   static_assert(SS_HELPERS % CB == 0 && 2 * TC * NP % SS_HELPERS == 0, "a helper keeps to its channels");
-  extern __shared__ __align__(16) float ss_s[];  // two buffers, then y of two tiles [TC][CB]
-  float* y_s = ss_s + 2 * BUF;
+  extern __shared__ __align__(16) float ss_s[];  // a buffer per group, then as many tiles of y [TC][CB]
+  __shared__ __align__(8) unsigned long long bars[2 * SS_GROUPS];  // per buffer: a tile is there; it has been scanned
+  float* y_s = ss_s + SS_GROUPS * BUF;
   allow_dependents();
   const int tid = threadIdx.x, c0 = blockIdx.x * CB, s = blockIdx.y;
   const bool scans = tid < SCAN;
@@ -249,7 +237,7 @@ __global__ void __launch_bounds__(ss_scan_threads(L) + 2 * SS_HELPERS) selective
       a2[k] = live && n < p.N ? p.a2[(size_t)c * p.N + n] : 0.f;
     }
   }
-  const int pair = (tid - SCAN) / SS_HELPERS, helper = (tid - SCAN) % SS_HELPERS;  // of a helper
+  const int group = (tid - SCAN) / SS_HELPERS, helper = (tid - SCAN) % SS_HELPERS;  // of a helper
   const int q = scans ? 0 : (helper % LANES) * PV, k0 = scans ? 0 : helper / LANES;
   const bool q_ok = !scans && c0 + q < p.inner;
   float bias[PV], skip[PV];
@@ -268,6 +256,18 @@ __global__ void __launch_bounds__(ss_scan_threads(L) + 2 * SS_HELPERS) selective
   float* st = MODE == 0 ? p.state + (size_t)p.seq_slots[s] * p.state_stride : p.chunk_states + place * p.inner * p.N;
   st += (size_t)c * p.N;
   const int tiles = (n_tok + TC - 1) / TC;
+  if (tid == 0) {
+    for (int g = 0; g < SS_GROUPS; ++g) {
+      mbar_init(smem_u32(&bars[g]), SS_HELPERS);
+      mbar_init(smem_u32(&bars[SS_GROUPS + g]), SCAN / 32);
+    }
+    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+  }
+  // Packs of B and C: what lies behind N states of a row is never written again.
+  if (VEC && p.N < NP)
+    for (int idx = tid; idx < SS_GROUPS * 2 * TC * NP; idx += blockDim.x)
+      if ((idx & (NP - 1)) >= p.N) ss_s[(idx / (2 * TC * NP)) * BUF + 2 * TC * CB + idx % (2 * TC * NP)] = 0.f;
+  __syncthreads();
   if (scans) {
 #pragma unroll
     for (int k = 0; k < NS; ++k) {
@@ -275,54 +275,92 @@ __global__ void __launch_bounds__(ss_scan_threads(L) + 2 * SS_HELPERS) selective
       S[k] = MODE != 1 && live && n < p.N ? st[n] : 0.f;
     }
     float dt_sum = 0.f;
-    __syncthreads();  // the first tile is there
     for (int i = 0; i < tiles; ++i) {
-      const float* buf = ss_s + (i & 1) * BUF;
+      const int g_of = i % SS_GROUPS;
+      const float* buf = ss_s + g_of * BUF;
+      mbar_wait(smem_u32(&bars[g_of]), (uint32_t)(i / SS_GROUPS) & 1u, p.status);
       const float* dt_s = buf + ch;
       const float* dx_s = buf + TC * CB + ch;
       const float* bc_s = buf + 2 * TC * CB + r * NS;
-      float* y_out = y_s + (i & 1) * TC * CB + ch;
-      // A tile's sums stay in registers until its last token: a store among the loads of later tokens would hold
-      // them up (it could be to the same place).
+      float* y_out = y_s + g_of * TC * CB + ch;
+      // Four tokens at a time, in the order in which a warp should issue them: the next four's loads, this four's sums,
+      // the next four's decays.  A tile's sums stay in registers until its last token: a store among the loads of
+      // later tokens would hold them up (it could be to the same place).
       constexpr int OWN = L >= 4 ? 1 : 4 / L;
       float sums[TC / 4][OWN];
       int token = 0;
-#pragma unroll
-      for (int g = 0; g < TC; g += 4) {
-        float y[4];
+      float decay[4][NS], input[4][NS], cc[4][NS];
+      auto load = [&](int g, float (&dt)[4], float (&dx)[4], float (&b)[4][NS], float (&c)[4][NS]) {
 #pragma unroll
         for (int kk = 0; kk < 4; ++kk) {
           const int k = g + kk;
-          const float dt = dt_s[k * CB], dx = dx_s[k * CB];
-          if (MODE == 1) dt_sum += dt;
-          float b[NS], cc[NS];
+          dt[kk] = dt_s[k * CB], dx[kk] = dx_s[k * CB];
 #pragma unroll
           for (int j = 0; j < NS; j += 4) {
             const float4 bv = *reinterpret_cast<const float4*>(bc_s + k * 2 * NP + j);
-            b[j] = bv.x, b[j + 1] = bv.y, b[j + 2] = bv.z, b[j + 3] = bv.w;
+            b[kk][j] = bv.x, b[kk][j + 1] = bv.y, b[kk][j + 2] = bv.z, b[kk][j + 3] = bv.w;
             if (MODE != 1) {
               const float4 cv = *reinterpret_cast<const float4*>(bc_s + k * 2 * NP + NP + j);
-              cc[j] = cv.x, cc[j + 1] = cv.y, cc[j + 2] = cv.z, cc[j + 3] = cv.w;
+              c[kk][j] = cv.x, c[kk][j + 1] = cv.y, c[kk][j + 2] = cv.z, c[kk][j + 3] = cv.w;
             }
           }
+        }
+      };
+      auto weigh = [&](const float (&dt)[4], const float (&dx)[4], const float (&b)[4][NS]) {
+#pragma unroll
+        for (int kk = 0; kk < 4; ++kk) {
+          if (MODE == 1) dt_sum += dt[kk];
+#pragma unroll
+          for (int j = 0; j < NS; ++j) {
+            decay[kk][j] = pow2_for<T>(dt[kk] * a2[j]);
+            input[kk][j] = dx[kk] * b[kk][j];
+          }
+        }
+      };
+      {
+        float dt[4], dx[4], b[4][NS];
+        load(0, dt, dx, b, cc);
+        weigh(dt, dx, b);
+      }
+#pragma unroll
+      for (int g = 0; g < TC; g += 4) {
+        float dt[4], dx[4], b[4][NS], c_next[4][NS];
+        if (g + 4 < TC) load(g + 4, dt, dx, b, c_next);
+        float y[4];
+#pragma unroll
+        for (int kk = 0; kk < 4; ++kk) {
           float acc = 0.f;
 #pragma unroll
           for (int j = 0; j < NS; ++j) {
-            S[j] = fmaf(pow2_for<T>(dt * a2[j]), S[j], dx * b[j]);
-            if (MODE != 1) acc = fmaf(S[j], cc[j], acc);
+            S[j] = fmaf(decay[kk][j], S[j], input[kk][j]);
+            if (MODE != 1) acc = fmaf(S[j], cc[kk][j], acc);
           }
           y[kk] = acc;
         }
-        if (MODE != 1) {
-          // Two tokens stay with each lane of a pair, then one with each lane of four.
-          if (L >= 2) {
-            const bool up = (r & 1) != 0;
+        // Two tokens stay with each lane of a pair, then one with each lane of four.
+        float kept[2], given[2];
+        if (MODE != 1 && L >= 2) {
+          const bool up = (r & 1) != 0;
 #pragma unroll
-            for (int e = 0; e < 2; ++e) {
-              const float give = up ? y[e] : y[e + 2], keep = up ? y[e + 2] : y[e];
-              y[e] = keep + __shfl_xor_sync(0xffffffffu, give, 1);
-            }
-            token = up ? 2 : 0;
+          for (int e = 0; e < 2; ++e) {
+            given[e] = __shfl_xor_sync(0xffffffffu, up ? y[e] : y[e + 2], 1);
+            kept[e] = up ? y[e + 2] : y[e];
+          }
+          token = up ? 2 : 0;
+        }
+        if (g + 4 < TC) {
+          weigh(dt, dx, b);
+          if (MODE != 1) {
+#pragma unroll
+            for (int kk = 0; kk < 4; ++kk)
+#pragma unroll
+              for (int j = 0; j < NS; ++j) cc[kk][j] = c_next[kk][j];
+          }
+        }
+        if (MODE != 1) {
+          if (L >= 2) {
+#pragma unroll
+            for (int e = 0; e < 2; ++e) y[e] = kept[e] + given[e];
           }
           if (L >= 4) {
             const bool up = (r & 2) != 0;
@@ -344,7 +382,8 @@ __global__ void __launch_bounds__(ss_scan_threads(L) + 2 * SS_HELPERS) selective
 #pragma unroll
           for (int e = 0; e < OWN; ++e) y_out[(g + token + e) * CB] = sums[g / 4][e];
       }
-      __syncthreads();
+      __syncwarp();
+      if ((tid & 31) == 0) mbar_arrive(smem_u32(&bars[SS_GROUPS + g_of]));
     }
     if (MODE != 2 && live) {
 #pragma unroll
@@ -380,10 +419,6 @@ __global__ void __launch_bounds__(ss_scan_threads(L) + 2 * SS_HELPERS) selective
       pack_col[u] = j;
       pack_at[u] = at < packs ? k * 2 * NP + (j < p.N ? j : NP + j - p.N) : -1;
     }
-    // What lies behind N states of a row is never written again.
-    if (p.N < NP)
-      for (int idx = tid - SCAN; idx < 4 * TC * NP; idx += 2 * SS_HELPERS)
-        if ((idx & (NP - 1)) >= p.N) ss_s[(idx / (2 * TC * NP)) * BUF + 2 * TC * CB + idx % (2 * TC * NP)] = 0.f;
   }
   auto fetch = [&](int i) {
     const int i0 = i * TC;
@@ -410,7 +445,7 @@ __global__ void __launch_bounds__(ss_scan_threads(L) + 2 * SS_HELPERS) selective
   };
   auto put = [&](int i) {
     const int i0 = i * TC;
-    float* buf = ss_s + (i & 1) * BUF;
+    float* buf = ss_s + group * BUF;
 #pragma unroll
     for (int u = 0; u < CH_PER; ++u) {
       const int k = k0 + u * STEP;
@@ -455,33 +490,26 @@ __global__ void __launch_bounds__(ss_scan_threads(L) + 2 * SS_HELPERS) selective
         float y[PV];
 #pragma unroll
         for (int e = 0; e < PV; ++e)
-          y[e] = fmaf(skip[e], past_x[u].get(e), y_s[(i & 1) * TC * CB + k * CB + q + e]) * silu_for<T>(past_z[u].get(e));
+          y[e] = fmaf(skip[e], past_x[u].get(e), y_s[group * TC * CB + k * CB + q + e]) * silu_for<T>(past_z[u].get(e));
         Pair::store(out + (size_t)(i * TC + k) * p.out_stride, y);
       }
     }
   };
-  // A pair's turn: the sums of its tile before, then its next tile into the other buffer, then the loads of the one
-  // after that.  (A tile of a token behind the end has dt = dx = 0: what B and C hold there does not matter.)
-  auto turn = [&](int i) {  // tile i is scanned; i + 1 is put in place, i - 1 is done
-    if (MODE != 1 && i > 0) finish(i - 1);
-    if (i + 1 < tiles) {
-      put(i + 1);
+  // (A token behind the end has dt = dx = 0: what B and C hold there does not matter.)
+  const uint32_t there = smem_u32(&bars[group]), scanned = smem_u32(&bars[SS_GROUPS + group]);
+  if (group < tiles) fetch(group);
+  for (int t = group; t < tiles; t += SS_GROUPS) {
+    put(t);
+    mbar_arrive(there);
 #pragma unroll
-      for (int u = 0; u < CH_PER; ++u) {
-        past_x[u] = in_x[u];
-        if (MODE != 1) past_z[u] = in_z[u];
-      }
-      if (i + 3 < tiles) fetch(i + 3);
+    for (int u = 0; u < CH_PER; ++u) {
+      past_x[u] = in_x[u];
+      if (MODE != 1) past_z[u] = in_z[u];
     }
-  };
-  if (pair < tiles) fetch(pair);
-  if (pair == 0) turn(-1);
-  __syncthreads();
-  for (int i = 0; i < tiles; ++i) {
-    if (((i + 1) & 1) == pair) turn(i);
-    __syncthreads();
+    if (t + SS_GROUPS < tiles) fetch(t + SS_GROUPS);
+    mbar_wait(scanned, (uint32_t)(t / SS_GROUPS) & 1u, p.status);
+    if (MODE != 1) finish(t);
   }
-  if (MODE != 1 && ((tiles - 1) & 1) == pair) finish(tiles - 1);
 }
 
 // Per sequence: the states its chunks start from, in order (each in the place of the chunk's own last state), and
@@ -642,17 +670,16 @@ VX_API int vx_conv_act(const void* x, int dtype, long long x_stride, int channel
                        cudaStream_t stream) {
   if (num_seqs <= 0 || channels <= 0 || longest <= 0) return 0;
   if (taps < 1 || num_seqs > 65535) return (int)cudaErrorInvalidValue;
-  const int pack = dtype == VX_DTYPE_F32 ? 4 : 8;
-  const bool vec = channels % pack == 0 && x_stride % pack == 0 && out_stride % pack == 0 &&
-                   ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(out)) & 15) == 0;
+  const bool pairs = channels % 2 == 0 && x_stride % 2 == 0 && out_stride % 2 == 0 &&
+                     ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(out)) & 7) == 0;
 #define VX_CONV_LAUNCH(T, V)                                                                                           \
   launch_conv_act<T, V>(x, x_stride, channels, taps, w_t, bias, state, state_stride, out, out_stride, q_start, q_len, \
                         seq_slots, num_seqs, longest, act, stream)
   if (dtype == VX_DTYPE_F32) {
-    if (vec) VX_CONV_LAUNCH(float, 4);
+    if (pairs) VX_CONV_LAUNCH(float, 2);
     else VX_CONV_LAUNCH(float, 1);
   } else {
-    if (vec) VX_CONV_LAUNCH(__nv_bfloat16, 8);
+    if (pairs) VX_CONV_LAUNCH(__nv_bfloat16, 2);
     else VX_CONV_LAUNCH(__nv_bfloat16, 1);
   }
 #undef VX_CONV_LAUNCH
@@ -661,8 +688,8 @@ VX_API int vx_conv_act(const void* x, int dtype, long long x_stride, int channel
 
 template <typename T, int L, int NS, bool VEC>
 static int launch_selective_scan(const SelectiveScan& p, int num_seqs, int num_tokens, cudaStream_t stream) {
-  constexpr int THREADS = ss_scan_threads(L) + 2 * SS_HELPERS, CB = ss_scan_threads(L) / L, NP = L * NS, TC = ss_tile(L, NP);
-  constexpr size_t smem = sizeof(float) * 2 * (3 * TC * CB + 2 * TC * NP);
+  constexpr int THREADS = ss_scan_threads(L) + SS_GROUPS * SS_HELPERS, CB = ss_scan_threads(L) / L, NP = L * NS, TC = ss_tile(L, NP);
+  constexpr size_t smem = sizeof(float) * SS_GROUPS * (3 * TC * CB + 2 * TC * NP);
   static bool configured = false;
   if (smem > 48 * 1024 && !configured) {
     cudaError_t e = cudaFuncSetAttribute(selective_scan_kernel<T, L, NS, 0, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -727,12 +754,13 @@ VX_API int vx_selective_scan(const void* x, int dtype, long long x_stride, const
                              const float* d_skip, const void* z, long long z_stride, void* out, long long out_stride,
                              float* state, long long state_stride, int inner, int N, int chunk, float* chunk_states,
                              float* chunk_dt, const int* q_start, const int* q_len, const int* seq_slots, int num_seqs,
-                             int num_tokens, cudaStream_t stream) {
+                             int num_tokens, int* status, cudaStream_t stream) {
   if (num_seqs <= 0 || num_tokens <= 0) return 0;
   if (inner <= 0 || N <= 0 || N > 512 || num_seqs > 65535) return (int)cudaErrorInvalidValue;
   if (chunk_states == nullptr || chunk_dt == nullptr) chunk = 0;
   const SelectiveScan p = {x, x_stride, dt, dt_stride, dt_bias, a2, bc, bc_stride, d_skip, z, z_stride, out, out_stride,
-                           state, state_stride, inner, N, chunk, q_start, q_len, seq_slots, chunk_states, chunk_dt};
+                           state, state_stride, inner, N, chunk, q_start, q_len, seq_slots, chunk_states, chunk_dt,
+                           status};
 #define VX_SCAN_CALL(L, NS) VX_BY_DTYPE(dtype, return (choose_selective_scan<T, L, NS>(p, num_seqs, num_tokens, stream)))
   VX_SELECTIVE_SIZES(VX_SCAN_CALL)
 #undef VX_SCAN_CALL
@@ -759,7 +787,7 @@ VX_API int vx_selective_step(const void* x, int dtype, long long x_stride, const
   if (num_seqs <= 0) return 0;
   if (inner <= 0 || N <= 0 || N > 512 || rank <= 0 || num_seqs > 65535) return (int)cudaErrorInvalidValue;
   const SelectiveScan p = {x, x_stride, nullptr, 0, dt_bias, a2, nullptr, low_stride, d_skip, z, z_stride, out, out_stride,
-                           state, state_stride, inner, N, 0, q_start, nullptr, seq_slots, nullptr, nullptr};
+                           state, state_stride, inner, N, 0, q_start, nullptr, seq_slots, nullptr, nullptr, nullptr};
 #define VX_STEP_CALL(L, NS) VX_BY_DTYPE(dtype, return (launch_selective_step<T, L, NS>(p, low, w_dt, rank, num_seqs, stream)))
   VX_SELECTIVE_SIZES(VX_STEP_CALL)
 #undef VX_STEP_CALL

@@ -206,7 +206,7 @@ def mixers():
         lib.vx_selective_block_channels.argtypes = [_c_int]
         lib.vx_selective_scan.argtypes = [
             _ptr, _c_int, _c_ll, _ptr, _c_ll, _ptr, _ptr, _ptr, _c_ll, _ptr, _ptr, _c_ll, _ptr, _c_ll, _ptr, _c_ll, _c_int,
-            _c_int, _c_int, _ptr, _ptr, _ptr, _ptr, _ptr, _c_int, _c_int, _ptr,
+            _c_int, _c_int, _ptr, _ptr, _ptr, _ptr, _ptr, _c_int, _c_int, _ptr, _ptr,
         ]
         lib.vx_selective_step.argtypes = [
             _ptr, _c_int, _c_ll, _ptr, _c_ll, _ptr, _c_int, _ptr, _ptr, _ptr, _ptr, _c_ll, _ptr, _c_ll, _ptr, _c_ll,
@@ -1848,7 +1848,7 @@ def selective_chunk(num_tokens: int, num_seqs: int, inner: int, states: int) -> 
     return max(64, -(-num_tokens * blocks // (6 * 148 * 16)) * 16)
 
 
-def selective_scan(x, dt, dt_bias, a2, bc, d_skip, z, out, state, q_start, q_len, seq_slots, num_seqs, num_tokens,
+def selective_scan(x, dt, dt_bias, a2, bc, d_skip, z, out, state, q_start, q_len, seq_slots, num_seqs, num_tokens, status,
                    chunk=0, chunk_states=None, chunk_dt=None) -> None:
     """Per channel c and state n: ``S <- exp(dt A) S + dt x B``, ``out = (sum_n S C + D x) * silu(z)`` with ``dt =
     softplus(dt + dt_bias)`` (``dt`` float32 logits) and ``a2 = A log2(e)`` float32 [inner, states]; ``bc`` rows hold B |
@@ -1856,6 +1856,7 @@ def selective_scan(x, dt, dt_bias, a2, bc, d_skip, z, out, state, q_start, q_len
     tokens side by side, with float32 scratch ``chunk_states`` ((num_tokens // chunk + num_seqs + 1) * inner * states
     values) and ``chunk_dt`` (as many times inner)."""
     inner, states = _selective_check(x, dt_bias, a2, d_skip, z, out, state)
+    _need(status, torch.int32, "status")
     if dt.dtype != torch.float32 or dt.shape[1] != inner or bc.dtype != x.dtype or bc.shape[1] != 2 * states:
         raise ValueError("selective_scan: dt or bc do not match")
     if chunk > 0:
@@ -1868,7 +1869,7 @@ def selective_scan(x, dt, dt_bias, a2, bc, d_skip, z, out, state, q_start, q_len
         _p(x), _code(x.dtype), _pitched(x, "x"), _p(dt), _pitched(dt, "dt"), _p(dt_bias), _p(a2), _p(bc), _pitched(bc, "bc"),
         _p(d_skip), _p(z), _pitched(z, "z"), _p(out), _pitched(out, "out"), _p(state), state.stride(0), inner, states,
         int(chunk), _p(chunk_states) if chunk > 0 else None, _p(chunk_dt) if chunk > 0 else None, _p(q_start), _p(q_len),
-        _p(seq_slots), num_seqs, num_tokens, _stream()), "selective_scan")
+        _p(seq_slots), num_seqs, num_tokens, _p(status), _stream()), "selective_scan")
 
 
 def selective_step(x, low, w_dt, dt_bias, a2, d_skip, z, out, state, q_start, seq_slots, num_seqs) -> bool:

@@ -531,7 +531,7 @@ class SelectiveScan(Mixer):
                 chunk_states = ws.get(f"selective.chunk_states{I}_{N}", (places * I * N,), torch.float32)
                 chunk_dt = ws.get(f"selective.chunk_dt{I}", (places * I,), torch.float32)
             kernels.selective_scan(u[:, :I], dt[:, :I], self.dt_bias, self.a2, low[:, R : R + 2 * N], self.d_skip, z, y[:, :I],
-                                   state[:, : self.state_elems], ctx.q_start, ctx.q_len, ctx.seq_slots, ctx.num_seqs, T,
+                                   state[:, : self.state_elems], ctx.q_start, ctx.q_len, ctx.seq_slots, ctx.num_seqs, T, ctx.status,
                                    chunk=chunk, chunk_states=chunk_states, chunk_dt=chunk_dt)
         return product_of(y, self.w_out, ctx, T)
 
